@@ -103,6 +103,7 @@ class ModelPlan:
     # residual streams a token (the blocks' arrangement reads and writes all of them; they start as
     # copies of the embedding and the last norm reads their sum)
     streams: int = 1
+    embedding_scale: float = 1.0                                # the stream starts as embedding * embedding_scale
     logit_softcap: float = 0.0                                  # > 0: logits <- cap * tanh(logits / cap)
 
 

@@ -12,7 +12,8 @@
 // Options beside the reference's mathematics: `slopes` (one per query head) takes
 // slope_h * (p - j) off the score of key j; `keep_first` keeps the first keys of a request
 // visible when the window has passed them (at their true positions); `gate` multiplies head h's
-// output by sigmoid(gate[t, h]).
+// output by sigmoid(gate[t, h]); `sig_bias` (one per query head) replaces the softmax by
+// sigmoid(score + sig_bias_h), a key's own weight, not normalised over keys.
 #include "common.cuh"
 
 namespace nf {
@@ -27,7 +28,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_row_stride,
                                const int* __restrict__ row_seg, T* __restrict__ out, int Hq,
                                int Hkv, int D, int page_size, int num_pages, int window,
                                float scale, const float* __restrict__ slopes, int keep_first,
-                               const float* __restrict__ gate, int gate_ld) {
+                               const float* __restrict__ gate, int gate_ld, const float* __restrict__ sig_bias) {
   extern __shared__ float q_smem[];          // [4 warps][D]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
@@ -82,14 +83,19 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_row_stride,
         s = dot * scale - slope * (float)(pos - j);
       }
     }
-    const float m_new = fmaxf(m, warp_max(s));
-    if (m_new == -INFINITY) continue;      // no visible key in this block (cannot happen for j0 <= pos)
-    const float p = (s == -INFINITY) ? 0.f : expf(s - m_new);
-    const float alpha = (m == -INFINITY) ? 0.f : expf(m - m_new);
-    l = l * alpha + warp_sum(p);
-    m = m_new;
+    float p;
+    if (sig_bias) {
+      p = (s == -INFINITY) ? 0.f : 1.f / (1.f + expf(-(s + sig_bias[h])));
+    } else {
+      const float m_new = fmaxf(m, warp_max(s));
+      if (m_new == -INFINITY) continue;    // no visible key in this block (cannot happen for j0 <= pos)
+      p = (s == -INFINITY) ? 0.f : expf(s - m_new);
+      const float alpha = (m == -INFINITY) ? 0.f : expf(m - m_new);
+      l = l * alpha + warp_sum(p);
+      m = m_new;
 #pragma unroll
-    for (int i = 0; i < kMaxDimsPerLane; ++i) acc[i] *= alpha;
+      for (int i = 0; i < kMaxDimsPerLane; ++i) acc[i] *= alpha;
+    }
     const int nkeys = min(32, last - j0 + 1);
     for (int jj = 0; jj < nkeys; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -104,7 +110,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_row_stride,
     }
   }
   }
-  float inv_l = l > 0.f ? 1.f / l : 0.f;
+  float inv_l = sig_bias ? 1.f : (l > 0.f ? 1.f / l : 0.f);
   if (gate) inv_l *= 1.f / (1.f + expf(-gate[(size_t)t * gate_ld + h]));
   T* o = out + (size_t)t * Hq * D + (size_t)h * D;
 #pragma unroll
@@ -124,15 +130,15 @@ extern "C" int nf_paged_attention_generic(const void* qkv, int q_row_stride, con
                                           int T, int Hq, int Hkv, int D, int page_size,
                                           int num_pages, int window, float scale, int dtype,
                                           const float* slopes, int keep_first, const float* gate, int gate_ld,
-                                          cudaStream_t stream) {
+                                          const float* sig_bias, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: bad sizes T=%d Hq=%d Hkv=%d", T, Hq, Hkv);
   NF_REQUIRE(D >= 1 && D <= 256, "attention: head_dim %d must lie in [1, 256]", D);
   dim3 grid(T, (Hq + 3) / 4);
   const size_t smem = 4 * D * sizeof(float);
   if (dtype == kF32)
-    paged_attention_generic_kernel<float><<<grid, 128, smem, stream>>>((const float*)qkv, q_row_stride, (const float*)pages, block_table, bt_width, positions, row_seg, (float*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld);
+    paged_attention_generic_kernel<float><<<grid, 128, smem, stream>>>((const float*)qkv, q_row_stride, (const float*)pages, block_table, bt_width, positions, row_seg, (float*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, sig_bias);
   else
-    paged_attention_generic_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width, positions, row_seg, (__nv_bfloat16*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld);
+    paged_attention_generic_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width, positions, row_seg, (__nv_bfloat16*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, sig_bias);
   return check_launch("paged_attention_generic");
 }

@@ -16,7 +16,8 @@
 // Options: `keep_first` keeps a request's first keys visible when the window has passed them (the
 // aligned blocks that hold them are walked first, then the window's); `slopes` takes
 // slope_h * (p - j) off head h's score of key j; `gate` multiplies head h's output by
-// sigmoid(gate[row, h]).
+// sigmoid(gate[row, h]).  The SIGMOID form replaces the softmax by weights sigmoid(score + sig_bias[h])
+// that are not normalised over keys: no maximum, no denominator, shares of a split row simply add.
 // Steps of single rows (decode) may split a row's key blocks over several CTAs: the blocks of kept
 // first keys are one share, and every aligned group of a few window blocks (four: 256 keys, by
 // absolute position) another; each CTA leaves its unnormalised sum, maximum and denominator, and a
@@ -59,7 +60,7 @@ __device__ __forceinline__ unsigned pf_pack(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 __global__ void __launch_bounds__(kThreads)
 prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride,
                          const __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table,
@@ -68,7 +69,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
                          int page_size, int num_pages, int window, float scale,
                          const float* __restrict__ slopes, int keep_first, const float* __restrict__ gate,
                          int gate_ld, int n_shares, float* __restrict__ part_o, float* __restrict__ part_ml,
-                         int kSplitBlocks) {
+                         int kSplitBlocks, const float* __restrict__ sig_bias) {
   constexpr int DS = D + 8;             // padded row stride in elements
   constexpr int LPR = D / 8;            // 16-byte pieces per row
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -148,7 +149,9 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
   for (int n = 0; n < D / 8; ++n)
 #pragma unroll
     for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  // (the sigmoid form keeps no maximum and no denominator: its shares carry the maximum 0)
+  float m_run[2] = {SIGMOID ? 0.f : -INFINITY, SIGMOID ? 0.f : -INFINITY}, l_run[2] = {SIGMOID ? 1.f : 0.f, SIGMOID ? 1.f : 0.f};
+  const float sb2 = SIGMOID ? sig_bias[h] * kLog2e : 0.f;
   // this thread's two query rows and their positions
   const int r_lo = warp * 16 + g, r_hi = r_lo + 8;
   const int p_lo = pos_first + r_lo, p_hi = pos_first + r_hi;
@@ -218,6 +221,13 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
           mx[i >> 1] = fmaxf(mx[i >> 1], v);
         }
     }
+    if constexpr (SIGMOID) {
+      // 2^inf = inf for a masked key: its weight is exactly zero
+#pragma unroll
+      for (int n = 0; n < kBKeys / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[n][i] = __fdividef(1.f, 1.f + exp2f(-(s[n][i] + sb2)));
+    } else {
     float alpha[2], m_use[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -248,6 +258,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
       o[n][0] *= alpha[0]; o[n][1] *= alpha[0];
       o[n][2] *= alpha[1]; o[n][3] *= alpha[1];
     }
+    }  // softmax
     // ---- O += P V ----------------------------------------------------------------------------------
 #pragma unroll
     for (int kk = 0; kk < kBKeys / 16; ++kk) {
@@ -284,7 +295,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
       if (tq == 0) { part_ml[slot * 2] = m_run[r]; part_ml[slot * 2 + 1] = l_run[r]; }
       continue;
     }
-    float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
+    float inv = SIGMOID ? 1.f : (l_run[r] > 0.f ? 1.f / l_run[r] : 0.f);
     if (gate) inv *= 1.f / (1.f + expf(-gate[(size_t)(row0 + row) * gate_ld + h]));
     __nv_bfloat16* dst = out + (size_t)(row0 + row) * Hq * D + (size_t)h * D;
 #pragma unroll
@@ -302,7 +313,7 @@ __global__ void split_rows_merge_kernel(const float* __restrict__ part_o, const 
                                         const int* __restrict__ positions, const int* __restrict__ tiles,
                                         __nv_bfloat16* __restrict__ out, int Hq, int D,
                                         int window, int keep_first, int n_shares, const float* __restrict__ gate,
-                                        int gate_ld, int kSplitBlocks) {
+                                        int gate_ld, int kSplitBlocks, int normalise) {
   const int t = tiles[4 * blockIdx.x + 1], h = blockIdx.y;      // a tile is one row: its first row
   chain_release_if_small();
   const int pos = positions[t];
@@ -322,7 +333,7 @@ __global__ void split_rows_merge_kernel(const float* __restrict__ part_o, const 
     const float mz = part_ml[(base + z) * 2];
     if (mz != -INFINITY) l += part_ml[(base + z) * 2 + 1] * exp2f(mz - m);
   }
-  float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = !normalise ? 1.f : (l > 0.f ? 1.f / l : 0.f);
   if (gate) inv *= 1.f / (1.f + expf(-gate[(size_t)t * gate_ld + h]));
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float acc = 0.f;
@@ -334,28 +345,28 @@ __global__ void split_rows_merge_kernel(const float* __restrict__ part_o, const 
   }
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 static int launch_prefill(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                           int bt_width, const int* positions, const int* seg_row0, const int* tiles,
                           int n_tiles, void* out, int Hq, int Hkv, int page_size, int num_pages, int window,
                           float scale, const float* slopes, int keep_first, const float* gate, int gate_ld,
-                          int n_shares, float* part_o, float* part_ml, cudaStream_t stream) {
+                          int n_shares, float* part_o, float* part_ml, const float* sig_bias, cudaStream_t stream) {
   const size_t smem = (size_t)(kBQ + 4 * kBKeys) * (D + 8) * sizeof(__nv_bfloat16);
   static bool set = false;
   if (smem > 48 * 1024 && !set) {
-    cudaFuncSetAttribute(prefill_attention_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(prefill_attention_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     set = true;
   }
   dim3 grid(n_tiles, Hq, n_shares > 0 ? n_shares : 1);
-  prefill_attention_kernel<D><<<grid, kThreads, smem, stream>>>(
+  prefill_attention_kernel<D, SIGMOID><<<grid, kThreads, smem, stream>>>(
       (const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width, positions,
       seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale, slopes, keep_first, gate,
-      gate_ld, n_shares, part_o, part_ml, g_split_blocks);
+      gate_ld, n_shares, part_o, part_ml, g_split_blocks, sig_bias);
   if (int rc = check_launch("prefill_attention")) return rc;
   if (n_shares > 0) {
     launch_chained(split_rows_merge_kernel, dim3(n_tiles, Hq), dim3(D >= 64 ? 64 : 32), 0, stream, (const float*)part_o,
                    (const float*)part_ml, positions, tiles, (__nv_bfloat16*)out, Hq, D, window, keep_first, n_shares, gate, gate_ld,
-                   g_split_blocks);
+                   g_split_blocks, SIGMOID ? 0 : 1);
     return check_launch("split_rows_merge");
   }
   return 0;
@@ -386,22 +397,26 @@ extern "C" int nf_set_attention_split_blocks(int n) {
 // tiles as (segment, first row), each at most 64 consecutive rows of one segment; the second may
 // be (-1, -1).  slopes float32 [Hq] or null; keep_first >= 0 (it counts only with a window); gate
 // float32 [T, gate_ld] (column h: head h's gate logit) or null.  n_shares > 0: every tile is one row, and a row's key blocks are split into shares (see the top of this file); n_shares must be at least
-// nf_prefill_attention_shares(window, longest context); part_o float32 [rows, Hq, n_shares, D], part_ml
+// nf_prefill_attention_shares(window, longest context); sig_bias float32 [Hq] or null: sigmoid weights in the softmax's
+// place (then without slopes); part_o float32 [rows, Hq, n_shares, D], part_ml
 // [rows, Hq, n_shares, 2].
 extern "C" int nf_prefill_attention_biased(const void* qkv, int q_row_stride, const void* pages,
                                            const int* block_table, int bt_width, const int* positions,
                                            const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
                                            int Hkv, int D, int page_size, int num_pages, int window, float scale,
                                            const float* slopes, int keep_first, const float* gate, int gate_ld,
-                                           int n_shares, float* part_o, float* part_ml, cudaStream_t stream) {
+                                           int n_shares, float* part_o, float* part_ml, const float* sig_bias,
+                                           cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   NF_REQUIRE(n_shares >= 0 && n_shares <= 65535 && (n_shares == 0 || (part_o && part_ml)),
              "prefill attention: split rows need their workspace");
   NF_REQUIRE(n_tiles > 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0 && Hq <= 65535, "prefill attention: bad sizes tiles=%d Hq=%d Hkv=%d", n_tiles, Hq, Hkv);
   NF_REQUIRE(q_row_stride % 8 == 0 && (uintptr_t)qkv % 16 == 0, "prefill attention: query rows must be 16-byte aligned");
   NF_REQUIRE(keep_first >= 0 && (!gate || gate_ld >= Hq), "prefill attention: bad options");
+  NF_REQUIRE(!(sig_bias && slopes), "prefill attention: sigmoid weights and slopes do not go together");
   if (window <= 0) keep_first = 0;
-#define NF_PF(DD) case DD: return launch_prefill<DD>(qkv, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, n_shares, part_o, part_ml, stream);
+#define NF_PF_CALL(DD, SG) launch_prefill<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, n_shares, part_o, part_ml, sig_bias, stream)
+#define NF_PF(DD) case DD: return sig_bias ? NF_PF_CALL(DD, true) : NF_PF_CALL(DD, false);
   switch (D) {
     NF_PF(16) NF_PF(32) NF_PF(48) NF_PF(64) NF_PF(80) NF_PF(96) NF_PF(112) NF_PF(128)
     default:
@@ -409,6 +424,7 @@ extern "C" int nf_prefill_attention_biased(const void* qkv, int q_row_stride, co
       return 1;
   }
 #undef NF_PF
+#undef NF_PF_CALL
 }
 
 extern "C" int nf_prefill_attention(const void* qkv, int q_row_stride, const void* pages,
@@ -418,5 +434,5 @@ extern "C" int nf_prefill_attention(const void* qkv, int q_row_stride, const voi
                                     cudaStream_t stream) {
   return nf_prefill_attention_biased(qkv, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles,
                                      n_tiles, out, Hq, Hkv, D, page_size, num_pages, window, scale, nullptr, 0, nullptr,
-                                     0, 0, nullptr, nullptr, stream);
+                                     0, 0, nullptr, nullptr, nullptr, stream);
 }

@@ -27,6 +27,9 @@
 //              shared memory in the swizzled K-major image; at the end of the tile O divided by
 //              the row sum is stored
 //
+// The SIGMOID form has weights sigmoid(score + sig_bias[h]) that are not normalised over keys: no maximum, no rescaling,
+// no sum; P = 1 / (1 + 2^-(s + b)) and O is stored as it stands.
+//
 // Everything between the roles goes through mbarriers; every wait is bounded: after a fixed
 // number of polls the kernel records a code in `g_fa_error`, tells its other warps to stop,
 // waits (bounded) for its own copies in flight, frees its tensor memory and returns.
@@ -101,13 +104,13 @@ __device__ __forceinline__ TileInfo tile_info(const int* tiles, int which, const
   return t;
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 __global__ void __launch_bounds__(kFaThreads, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             const int* __restrict__ block_table, int bt_width, const int* __restrict__ positions,
                             const int* __restrict__ seg_row0, const int* __restrict__ tiles,
                             __nv_bfloat16* __restrict__ out, int Hq, int Hkv, int page_size, int num_pages,
-                            int window, float scale) {
+                            int window, float scale, const float* __restrict__ sig_bias) {
   constexpr int ATOMS = D / 64;                   // 64-column swizzle atoms across the head
   constexpr int QB = ATOMS * kAtom;               // bytes of the Q tile, of a K block, of a V block
   extern __shared__ unsigned char smem_raw[];
@@ -289,6 +292,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int r = quad * 32 + lane;
     const unsigned lane_addr = (unsigned)(quad * 32) << 16;
     const float sc2 = scale * kLog2e;
+    const float sb2 = SIGMOID ? sig_bias[h] * kLog2e : 0.f;
     constexpr int HK = kKeys / 2;                    // score columns of this thread
     constexpr int HD = D / 2;                        // output columns of this thread
     int gs = 0, gp = 0, gq = 0;
@@ -323,8 +327,16 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&bars->s_empty[s]);           // the buffer may take the scores of block + 2
-        float mx;
-        {
+        float mx = 0.f;
+        if constexpr (SIGMOID) {
+          if (!all_visible) {
+#pragma unroll
+            for (int i = 0; i < HK; ++i) {
+              const bool vis = row_sees && (unsigned)(half * HK + i - j_lo) <= j_span;
+              u[i] = vis ? u[i] : 0xff800000u;                   // -inf: its weight is exactly zero
+            }
+          }
+        } else {
           float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};     // four chains, not one
           if (all_visible) {
 #pragma unroll
@@ -341,15 +353,18 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         // the row's maximum: the larger of the two halves (slots alternate with the block's parity,
         // so a fast thread cannot overwrite what its partner has yet to read)
-        float* slot = s_rowmax + (gs & 1) * 2 * kQ;
-        slot[half * kQ + r] = mx;
-        pair_sync();
-        mx = fmaxf(mx, slot[(half ^ 1) * kQ + r]) * sc2;         // sc2 > 0: the maximum of the scaled scores
+        if constexpr (!SIGMOID) {
+          float* slot = s_rowmax + (gs & 1) * 2 * kQ;
+          slot[half * kQ + r] = mx;
+          pair_sync();
+          mx = fmaxf(mx, slot[(half ^ 1) * kQ + r]) * sc2;       // sc2 > 0: the maximum of the scaled scores
+        }
         // the reference maximum: set by the first block with a visible key, raised only when a
         // score passes it by 2^8 (both threads of a row decide alike)
         float alpha = 1.f;
         bool raise = false;
-        if (!have) {                       // nothing visible so far (O's row and l are zero)
+        if (SIGMOID) {
+        } else if (!have) {                // nothing visible so far (O's row and l are zero)
           have = mx != -INFINITY;
           m_ref = have ? mx : 0.f;
         } else if (mx > m_ref + kRaise) {
@@ -359,7 +374,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         }
         // P and O are free once the product of the block before has run
         if (gp > 0 && !mbar_wait(&bars->p_free, (gp - 1) & 1, stop, 9, &g_fa_error)) { ok = false; break; }
-        if (__any_sync(0xffffffffu, raise)) {                   // the whole warp, each row by its own factor
+        if (!SIGMOID && __any_sync(0xffffffffu, raise)) {                   // the whole warp, each row by its own factor
           tc_fence_after();
 #pragma unroll 1
           for (int c = 0; c < HD / 32; ++c) {
@@ -382,7 +397,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         for (int q = 0; q < HK / 8; ++q) {
           float p[8];
 #pragma unroll
-          for (int i = 0; i < 8; ++i) p[i] = ex2(fmaf(__uint_as_float(u[8 * q + i]), sc2, -m_ref));
+          for (int i = 0; i < 8; ++i) {
+            if constexpr (SIGMOID) p[i] = __fdividef(1.f, 1.f + ex2(fmaf(__uint_as_float(u[8 * q + i]), -sc2, -sb2)));
+            else p[i] = ex2(fmaf(__uint_as_float(u[8 * q + i]), sc2, -m_ref));
+          }
           uint4 w;
           __nv_bfloat162 b0 = __floats2bfloat162_rn(p[0], p[1]), b1 = __floats2bfloat162_rn(p[2], p[3]);
           __nv_bfloat162 b2 = __floats2bfloat162_rn(p[4], p[5]), b3 = __floats2bfloat162_rn(p[6], p[7]);
@@ -401,10 +419,13 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       }
       if (!ok) break;
       // ---- the tile's rows: O / l ---------------------------------------------------------------------
-      s_rowsum[half * kQ + r] = l_run;
-      pair_sync();
-      const float l_row = s_rowsum[r] + s_rowsum[kQ + r];        // same order in both threads
-      pair_sync();                                               // both have read: the slots may be reused
+      float l_row = 1.f;
+      if constexpr (!SIGMOID) {
+        s_rowsum[half * kQ + r] = l_run;
+        pair_sync();
+        l_row = s_rowsum[r] + s_rowsum[kQ + r];                  // same order in both threads
+        pair_sync();                                             // both have read: the slots may be reused
+      }
       if (!mbar_wait(&bars->o_final, gq & 1, stop, 10, &g_fa_error)) { ok = false; break; }
       tc_fence_after();
       const float inv = l_row > 0.f ? 1.f / l_row : 0.f;
@@ -444,21 +465,22 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   }
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const int* block_table, int bt_width,
                       const int* positions, const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
-                      int Hkv, int page_size, int num_pages, int window, float scale, cudaStream_t stream) {
+                      int Hkv, int page_size, int num_pages, int window, float scale, const float* sig_bias,
+                      cudaStream_t stream) {
   constexpr int QB = (D / 64) * kAtom;
   const size_t smem = 1024 + (size_t)5 * QB + 2 * kAtom + sizeof(FaBarriers) + 6 * kQ * sizeof(float);
   static bool set = false;
   if (!set) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     NF_REQUIRE(e == cudaSuccess, "prefill attention: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     set = true;
   }
   dim3 grid(Hq, n_tiles);
-  launch_chained(prefill_attention_tc_kernel<D>, grid, dim3(kFaThreads), smem, stream, mq, mkv, block_table, bt_width,
-                 positions, seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale);
+  launch_chained(prefill_attention_tc_kernel<D, SIGMOID>, grid, dim3(kFaThreads), smem, stream, mq, mkv, block_table, bt_width,
+                 positions, seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias);
   return check_launch("prefill_attention_tc");
 }
 
@@ -479,12 +501,12 @@ extern "C" int nf_prefill_attention_tc_fits(int Hq, int Hkv, int D, int page_siz
 // bfloat16; head_dim 64 or 128; page size 16, 32, 64 or 128.  `tiles` is int32 [n_ctas, 2, 2]: for
 // every CTA two tiles as (segment, first row), each at most 128 consecutive rows of one segment;
 // the second may be (-1, -1).  qkv is [T, q_row_stride] with the queries in its first Hq * D
-// columns; out is [T, Hq * D].
+// columns; out is [T, Hq * D].  sig_bias float32 [Hq] or null: sigmoid weights in the softmax's place.
 extern "C" int nf_prefill_attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages,
                                        const int* block_table, int bt_width, const int* positions,
                                        const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
                                        int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                                       cudaStream_t stream) {
+                                       const float* sig_bias, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   NF_REQUIRE(n_tiles > 0 && n_tiles <= 65535 && T > 0, "prefill attention: bad sizes tiles=%d T=%lld", n_tiles, T);
   NF_REQUIRE(nf_prefill_attention_tc_fits(Hq, Hkv, D, page_size, num_pages), "prefill attention: sizes the tensor-core kernel does not take (Hq=%d Hkv=%d D=%d page=%d)", Hq, Hkv, D, page_size);
@@ -492,11 +514,10 @@ extern "C" int nf_prefill_attention_tc(const void* qkv, long long T, int q_row_s
   CUtensorMap mq, mkv;
   if (int rc = make_map(&mq, qkv, T, (long long)Hq * D, kQ, q_row_stride)) return rc;
   if (int rc = make_map(&mkv, pages, (long long)num_pages * 2 * Hkv * page_size, D, page_size)) return rc;
-  if (D == 64)
-    return launch_prefill_tc<64>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv,
-                                 page_size, num_pages, window, scale, stream);
-  return launch_prefill_tc<128>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv,
-                                page_size, num_pages, window, scale, stream);
+#define NF_TC(DD, SG) launch_prefill_tc<DD, SG>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, stream)
+  if (D == 64) return sig_bias ? NF_TC(64, true) : NF_TC(64, false);
+  return sig_bias ? NF_TC(128, true) : NF_TC(128, false);
+#undef NF_TC
 }
 
 // 0 if no tensor-core attention kernel has given up on a wait since the last call; else the code

@@ -13,7 +13,7 @@ namespace nf {
 
 template <typename T>
 __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                  float* __restrict__ out, int hidden, int vocab) {
+                                  float* __restrict__ out, int hidden, int vocab, float scale) {
   const int t = blockIdx.x;
   chain_wait();          // before the first write too: `out` may be memory that the kernel before still reads
   const int id = ids[t];
@@ -23,7 +23,7 @@ __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __rest
     return;
   }
   const T* row = table + (size_t)id * hidden;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_float(row[i]);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = to_float(row[i]) * scale;
 }
 
 // h[t] += delta[t] (if delta), out[t] = h[t] * rsqrt(mean(h[t]^2) + eps) * w.
@@ -302,13 +302,13 @@ static inline int row_threads(int n) {
 using namespace nf;
 
 extern "C" int nf_embed_rows(const void* table, const int* ids, float* out, int T, int hidden,
-                             int vocab, int dtype, cudaStream_t stream) {
+                             int vocab, float scale, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && hidden > 0 && vocab > 0, "embed_rows: bad sizes T=%d hidden=%d vocab=%d", T, hidden, vocab);
   if (dtype == kF32)
-    launch_chained(embed_rows_kernel<float>, dim3(T), dim3(row_threads(hidden)), 0, stream, (const float*)table, ids, out, hidden, vocab);
+    launch_chained(embed_rows_kernel<float>, dim3(T), dim3(row_threads(hidden)), 0, stream, (const float*)table, ids, out, hidden, vocab, scale);
   else
-    launch_chained(embed_rows_kernel<__nv_bfloat16>, dim3(T), dim3(row_threads(hidden)), 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, vocab);
+    launch_chained(embed_rows_kernel<__nv_bfloat16>, dim3(T), dim3(row_threads(hidden)), 0, stream, (const __nv_bfloat16*)table, ids, out, hidden, vocab, scale);
   return check_launch("embed_rows");
 }
 

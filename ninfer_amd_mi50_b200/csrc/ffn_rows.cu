@@ -43,6 +43,23 @@ __global__ void gelu_erf_kernel(T* __restrict__ x, size_t n) {
   }
 }
 
+// out = T(relu(z)^2), z the float32 sums of a product; W elements a thread
+template <typename T, int W>
+__global__ void relu_square_kernel(const float* __restrict__ z, T* __restrict__ out, size_t n) {
+  chain_wait(z);
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * W;
+  if (i >= n) return;
+  if constexpr (W == 4) {
+    float v[4];
+    load4(z + i, v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = relu_square(v[e]);
+    store4(out + i, v);
+  } else {
+    out[i] = from_float<T>(relu_square(z[i]));
+  }
+}
+
 // idx[t, j] = table[ids[t], j]: the experts of a token stand in a table by its id.  The loader has
 // checked that every entry names an expert and the step that every id lies in the table; an entry
 // that does not is read as expert 0 rather than followed.
@@ -91,6 +108,22 @@ extern "C" int nf_gelu_erf(void* x, long long n, int dtype, cudaStream_t stream)
   else
     launch_chained(gelu_erf_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)x, (size_t)n);
   return check_launch("gelu_erf");
+}
+
+extern "C" int nf_relu_square(const float* z, void* out, long long n, int dtype, cudaStream_t stream) {
+  if (n == 0) return 0;
+  NF_REQUIRE(n > 0, "relu_square: bad size %lld", n);
+  const bool vec = n % 4 == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)out % 16 == 0;
+  const long long units = vec ? n / 4 : n;
+  const dim3 grid((unsigned)((units + 255) / 256));
+  if (dtype == kF32) {
+    if (vec) launch_chained(relu_square_kernel<float, 4>, grid, dim3(256), 0, stream, z, (float*)out, (size_t)n);
+    else launch_chained(relu_square_kernel<float, 1>, grid, dim3(256), 0, stream, z, (float*)out, (size_t)n);
+  } else {
+    if (vec) launch_chained(relu_square_kernel<__nv_bfloat16, 4>, grid, dim3(256), 0, stream, z, (__nv_bfloat16*)out, (size_t)n);
+    else launch_chained(relu_square_kernel<__nv_bfloat16, 1>, grid, dim3(256), 0, stream, z, (__nv_bfloat16*)out, (size_t)n);
+  }
+  return check_launch("relu_square");
 }
 
 extern "C" int nf_table_route(const int* table, const int* ids, int* idx, int T, int k, int rows, int E,

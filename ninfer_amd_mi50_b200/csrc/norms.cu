@@ -95,6 +95,86 @@ __global__ void add_layernorm_kernel(float* __restrict__ h, const T* __restrict_
   }
 }
 
+// RMS norm in `groups` equal consecutive parts, fused with the residual sum of up to two contributions (a
+// mixer's and a feed-forward's that ran side by side):
+//   h[t] += d1[t] (+ d2[t]);  out[t] = part / sqrt(mean(part^2) + eps) * w   for each part of h[t].
+// With `rows`, row r reads h[rows[r]] / d1[rows[r]] / d2[rows[r]], writes out[r] and leaves h alone.
+// The row waits in shared memory between the passes; warps are dealt out evenly to the groups.
+// VEC: a group is a multiple of 4 elements and every operand's rows are aligned: runs of four an access.
+template <typename T, bool GATHER, bool VEC>
+__global__ void __launch_bounds__(256)
+add_group_rmsnorm_kernel(float* __restrict__ h, const T* __restrict__ d1, const T* __restrict__ d2,
+                         const int* __restrict__ rows, const float* __restrict__ w, float eps, int groups,
+                         T* __restrict__ out, int hidden) {
+  extern __shared__ __align__(16) float row[];      // [hidden], then partial sums [groups][warps a group], then inv [groups]
+  const int r = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
+  const int gs = hidden / groups;
+  const int wpg = nwarp > groups ? nwarp / groups : 1;      // warps a group
+  float* part = row + hidden;
+  float* inv = part + groups * wpg;
+  constexpr int W = VEC ? 4 : 1;
+  chain_release_if_small();
+  chain_wait(h, d1, d2, rows);
+  const int src = GATHER ? rows[r] : r;
+  float* hr = h + (size_t)src * hidden;
+  const T* a = d1 ? d1 + (size_t)src * hidden : nullptr;
+  const T* b = d2 ? d2 + (size_t)src * hidden : nullptr;
+  for (int i = threadIdx.x * W; i < hidden; i += blockDim.x * W) {
+    float v[W], x[W];
+    if constexpr (VEC) load4(hr + i, v); else v[0] = hr[i];
+    if (a) {
+      if constexpr (VEC) load4(a + i, x); else x[0] = to_float(a[i]);
+#pragma unroll
+      for (int e = 0; e < W; ++e) v[e] += x[e];
+    }
+    if (b) {
+      if constexpr (VEC) load4(b + i, x); else x[0] = to_float(b[i]);
+#pragma unroll
+      for (int e = 0; e < W; ++e) v[e] += x[e];
+    }
+    if (!GATHER && (a || b)) {
+      if constexpr (VEC) store4(hr + i, v); else hr[i] = v[0];
+    }
+#pragma unroll
+    for (int e = 0; e < W; ++e) row[i + e] = v[e];
+  }
+  __syncthreads();
+  for (int g = warp / wpg; g < groups; g += (nwarp + wpg - 1) / wpg) {
+    const int sub = warp - (warp / wpg) * wpg;
+    float ss = 0.f;
+    for (int i = (sub * 32 + lane) * W; i < gs; i += wpg * 32 * W) {
+      float v[W];
+      if constexpr (VEC) load4(row + g * gs + i, v); else v[0] = row[g * gs + i];
+#pragma unroll
+      for (int e = 0; e < W; ++e) ss = fmaf(v[e], v[e], ss);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) part[g * wpg + sub] = ss;
+  }
+  __syncthreads();
+  for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+    float ss = 0.f;
+    for (int s = 0; s < wpg; ++s) ss += part[g * wpg + s];
+    inv[g] = 1.f / sqrtf(ss / (float)gs + eps);
+  }
+  __syncthreads();
+  T* o = out + (size_t)r * hidden;
+  for (int i = threadIdx.x * W; i < hidden; i += blockDim.x * W) {
+    const float f = inv[i / gs];
+    if constexpr (VEC) {
+      float v[4], wv[4];
+      load4(row + i, v);
+      load4(w + i, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[e] = v[e] * f * wv[e];
+      store4(o + i, v);
+    } else {
+      o[i] = from_float<T>(row[i] * f * w[i]);
+    }
+  }
+}
+
 // out[t, 0:n] = x[t, col0:col0+n] * rsqrt(mean(x^2) + eps) * w   (w may be null: weight 1)
 template <typename T>
 __global__ void rms_norm_slice_kernel(const T* __restrict__ x, int ldx, int col0, int n,
@@ -151,13 +231,13 @@ __global__ void add_row_vector_kernel(float* __restrict__ h, const float* __rest
 // ([heads, T, n], what a batched product over heads leaves), out token by token.
 template <typename T>
 __global__ void heads_sigmoid_gate_kernel(const T* __restrict__ v, const T* __restrict__ g, int ldg, int gcol0,
-                                          T* __restrict__ out, int rows, int heads, int n) {
+                                          T* __restrict__ out, int rows, int heads, int n, int per_head) {
   const int t = blockIdx.x;
   chain_wait(v, g);
   const int width = heads * n;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     const int hd = c / n, i = c - hd * n;
-    const float gv = to_float(g[(size_t)t * ldg + gcol0 + c]);
+    const float gv = to_float(g[(size_t)t * ldg + gcol0 + (per_head ? hd : c)]);
     const float vv = to_float(v[((size_t)hd * rows + t) * n + i]);
     out[(size_t)t * width + c] = from_float<T>(vv * (1.f / (1.f + expf(-gv))));
   }
@@ -226,6 +306,36 @@ extern "C" int nf_add_layernorm(float* h, const void* delta, const int* rows, co
   return check_launch("add_layernorm");
 }
 
+// h float32 [T, hidden] (updated in place unless `rows`), d1 / d2 [T, hidden] in `dtype` or null, out [R, hidden].
+extern "C" int nf_add_group_rmsnorm(float* h, const void* d1, const void* d2, const int* rows, const float* w, float eps,
+                                    int groups, void* out, int R, int hidden, int dtype, cudaStream_t stream) {
+  if (R == 0) return 0;
+  NF_REQUIRE(R > 0 && hidden > 0 && w && groups >= 1 && hidden % groups == 0, "add_group_rmsnorm: %d groups of a row of %d", groups, hidden);
+  const size_t el = dtype == kF32 ? 4 : 2;
+  const bool vec = (hidden / groups) % 4 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+                   (uintptr_t)out % (4 * el) == 0 && (uintptr_t)d1 % (4 * el) == 0 && (uintptr_t)d2 % (4 * el) == 0;
+  int th = 64;
+  while (th < (vec ? hidden / 4 : hidden) && th < 256) th <<= 1;
+  const int nwarp = th / 32, wpg = nwarp > groups ? nwarp / groups : 1;
+  const size_t smem = ((size_t)hidden + (size_t)groups * (wpg + 1)) * sizeof(float);
+  NF_REQUIRE(smem <= 200 * 1024, "add_group_rmsnorm: a row of %d does not fit shared memory", hidden);
+#define NF_GN(TT, GA, VE)                                                                                             \
+  do {                                                                                                                \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(add_group_rmsnorm_kernel<TT, GA, VE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    launch_chained(add_group_rmsnorm_kernel<TT, GA, VE>, dim3(R), dim3(th), smem, stream, h, (const TT*)d1,           \
+                   (const TT*)d2, rows, w, eps, groups, (TT*)out, hidden);                                            \
+  } while (0)
+#define NF_GN2(TT)                                                                                                    \
+  do {                                                                                                                \
+    if (rows) { if (vec) NF_GN(TT, true, true); else NF_GN(TT, true, false); }                                        \
+    else { if (vec) NF_GN(TT, false, true); else NF_GN(TT, false, false); }                                           \
+  } while (0)
+  if (dtype == kF32) NF_GN2(float); else NF_GN2(__nv_bfloat16);
+#undef NF_GN2
+#undef NF_GN
+  return check_launch("add_group_rmsnorm");
+}
+
 extern "C" int nf_rms_norm_slice(const void* x, int ldx, int col0, int n, const float* w, float eps, void* out,
                                  int ldo, int R, int dtype, cudaStream_t stream) {
   if (R == 0) return 0;
@@ -261,14 +371,15 @@ extern "C" int nf_add_row_vector(float* h, const float* vec, int R, int hidden, 
   return check_launch("add_row_vector");
 }
 
+// per_head != 0: the gate has one logit a head (column gcol0 + head) instead of one an element
 extern "C" int nf_heads_sigmoid_gate(const void* v, const void* g, int ldg, int gcol0, void* out, int R, int heads,
-                                     int n, int dtype, cudaStream_t stream) {
+                                     int n, int per_head, int dtype, cudaStream_t stream) {
   if (R == 0) return 0;
-  NF_REQUIRE(heads > 0 && n > 0 && gcol0 >= 0 && gcol0 + heads * n <= ldg, "heads_sigmoid_gate: bad sizes");
+  NF_REQUIRE(heads > 0 && n > 0 && gcol0 >= 0 && gcol0 + heads * (per_head ? 1 : n) <= ldg, "heads_sigmoid_gate: bad sizes");
   if (dtype == kF32)
-    launch_chained(heads_sigmoid_gate_kernel<float>, dim3(R), dim3(256), 0, stream, (const float*)v, (const float*)g, ldg, gcol0, (float*)out, R, heads, n);
+    launch_chained(heads_sigmoid_gate_kernel<float>, dim3(R), dim3(256), 0, stream, (const float*)v, (const float*)g, ldg, gcol0, (float*)out, R, heads, n, per_head);
   else
-    launch_chained(heads_sigmoid_gate_kernel<__nv_bfloat16>, dim3(R), dim3(256), 0, stream, (const __nv_bfloat16*)v, (const __nv_bfloat16*)g, ldg, gcol0, (__nv_bfloat16*)out, R, heads, n);
+    launch_chained(heads_sigmoid_gate_kernel<__nv_bfloat16>, dim3(R), dim3(256), 0, stream, (const __nv_bfloat16*)v, (const __nv_bfloat16*)g, ldg, gcol0, (__nv_bfloat16*)out, R, heads, n, per_head);
   return check_launch("heads_sigmoid_gate");
 }
 

@@ -8,7 +8,8 @@
 // Cache page layout: [2 (k, v)][kv_heads][page_size][head_dim], as rope_append.cu writes it.
 //
 // A second kernel serves an attention with values of their own and a rotation after the same
-// whole-projection norms (in either page layout), and a third its elementwise output gate.
+// whole-projection norms or none (in either page layout; the values may be turned as well), a third its
+// elementwise output gate, and a fourth turns attention outputs back.
 #define NF_CHAIN_CLASS 4
 #include "common.cuh"
 
@@ -66,9 +67,13 @@ qk_whole_norm_append_kernel(const float* __restrict__ proj, int ld, int q_col0, 
 // `rot` dimensions of every q and k head turned by the row's position (pair (i, i + rot/2), angle
 // pos * inv_freq[i] in float32), cosine and sine both times `mag`; q goes out in the cache's type, the
 // key and the value (bias added) into the request's page.  Two page layouts:
-//   rows == 0: [2 (k, v)][kv_heads][page_size][D] (needs Dv == D), what the flash and decode kernels read;
+//   rows == 0: [2 (k, v)][kv_heads][page_size][P], what the flash and decode kernels read; P >= D and P >= Dv, the
+//   rest of a key, a value and a query (rows of Hq * P) is zero, so that sizes those kernels do not take, or that
+//   differ, can be widened to one that they take;
 //   rows == 1: [page_size][kv_heads * D | kv_heads * Dv], one row a token, for key and value sizes that differ.
 // Hkv == 0: a layer that reads another layer's keys brings queries only.
+// Further forms: wq null - no norms; interleaved - pairs (2i, 2i + 1) instead of (i, i + rot/2); v_freq - the value is
+// turned too, over all its Dv dimensions in the same layout of pairs, pair m by pos * v_freq[m] (no magnitude).
 // The row's normed values wait in shared memory (float32) between the two passes.
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -79,14 +84,17 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
                               float mag, const int* __restrict__ positions, const int* __restrict__ row_seg,
                               T* __restrict__ q_out, int Hq, int Hkv, int D, int Dv, T* __restrict__ pages,
                               const int* __restrict__ block_table, int bt_width, int page_size, int num_pages,
-                              int rows_layout) {
-  extern __shared__ __align__(16) float y[];   // [Hq * D + Hkv * D], then cosine and sine of the row's rot / 2 angles
+                              int rows_layout, int P, int interleaved, const float* __restrict__ v_freq) {
+  // [Hq * D + Hkv * D], cosine and sine of the row's rot / 2 angles, and of its Dv / 2 angles if values are turned
+  extern __shared__ __align__(16) float y[];
   __shared__ float red[33];
   const int t = blockIdx.x;
   const int QW = Hq * D, KW = Hkv * D;
   const int half = rot / 2;
   float* cs_s = y + QW + KW;
   float* sn_s = cs_s + half;
+  float* vcs_s = sn_s + half;
+  float* vsn_s = vcs_s + Dv / 2;
   chain_release_if_small();
   // the angles depend on the position alone (a step's input, not the kernel before's output): all heads share them
   const int pos = positions[t];
@@ -96,6 +104,13 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
     cs_s[u] = cs * mag;
     sn_s[u] = sn * mag;
   }
+  if (v_freq)
+    for (int u = threadIdx.x; u < Dv / 2; u += blockDim.x) {
+      float sn, cs;
+      sincosf((float)pos * v_freq[u], &sn, &cs);
+      vcs_s[u] = cs;
+      vsn_s[u] = sn;
+    }
   chain_wait(proj);
   const float* row = proj + (size_t)t * ld;
   float sq = 0.f, sk = 0.f;
@@ -128,10 +143,12 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
       sk = fmaf(v, v, sk);
     }
   }
-  const float inv_q = 1.f / sqrtf(block_sum(sq, red) / (float)QW + eps);
-  const float inv_k = KW ? 1.f / sqrtf(block_sum(sk, red) / (float)KW + eps) : 0.f;
-  for (int i = threadIdx.x; i < QW; i += blockDim.x) y[i] = y[i] * inv_q * wq[i];
-  for (int i = threadIdx.x; i < KW; i += blockDim.x) y[QW + i] = y[QW + i] * inv_k * wk[i];
+  if (wq) {
+    const float inv_q = 1.f / sqrtf(block_sum(sq, red) / (float)QW + eps);
+    const float inv_k = KW ? 1.f / sqrtf(block_sum(sk, red) / (float)KW + eps) : 0.f;
+    for (int i = threadIdx.x; i < QW; i += blockDim.x) y[i] = y[i] * inv_q * wq[i];
+    for (int i = threadIdx.x; i < KW; i += blockDim.x) y[QW + i] = y[QW + i] * inv_k * wk[i];
+  }
   __syncthreads();
   T* krow = nullptr;                           // where head 0's key of this token starts
   size_t k_head_stride = 0, v_head_stride = 0;
@@ -146,8 +163,8 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
         vrow = krow + (size_t)Hkv * D;
         k_head_stride = D; v_head_stride = Dv;
       } else {
-        krow = pages + ((size_t)page * 2 * Hkv * page_size + in_page) * D;
-        k_head_stride = v_head_stride = (size_t)page_size * D;
+        krow = pages + ((size_t)page * 2 * Hkv * page_size + in_page) * P;
+        k_head_stride = v_head_stride = (size_t)page_size * P;
         vrow = krow + (size_t)Hkv * k_head_stride;
       }
     }
@@ -158,27 +175,97 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
   for (int hh = warp; hh < Hq + Hkv; hh += nwarp) {       // a warp a head: q heads first, then k heads, as they lie in y
     const bool is_q = hh < Hq;
     const float* yy = y + (size_t)hh * D;
-    T* dst = is_q ? q_out + (size_t)t * QW + (size_t)hh * D
+    T* dst = is_q ? q_out + ((size_t)t * Hq + hh) * P
                   : (krow ? krow + (size_t)(hh - Hq) * k_head_stride : nullptr);
     if (!dst) continue;
     for (int u = lane; u < units; u += 32) {
       if (u < half) {
-        const float a = yy[u], b = yy[u + half];
+        const int i0 = interleaved ? 2 * u : u, i1 = interleaved ? 2 * u + 1 : u + half;
+        const float a = yy[i0], b = yy[i1];
         const float sn = sn_s[u], cs = cs_s[u];
-        dst[u] = from_float<T>(a * cs - b * sn);
-        dst[u + half] = from_float<T>(b * cs + a * sn);
+        dst[i0] = from_float<T>(a * cs - b * sn);
+        dst[i1] = from_float<T>(b * cs + a * sn);
       } else {
         const int d = rot + (u - half);
         dst[d] = from_float<T>(yy[d]);
       }
     }
+    if (is_q || !rows_layout)
+      for (int d = D + lane; d < P; d += 32) dst[d] = from_float<T>(0.f);
   }
   if (vrow) {
-    for (int head = warp; head < Hkv; head += nwarp)
-      for (int d = lane; d < Dv; d += 32) {
-        const int i = head * Dv + d;
-        vrow[(size_t)head * v_head_stride + d] = from_float<T>(row[v_col0 + i] + (bias_v ? bias_v[i] : 0.f));
+    const int vhalf = v_freq ? Dv / 2 : 0;
+    for (int head = warp; head < Hkv; head += nwarp) {
+      T* dst = vrow + (size_t)head * v_head_stride;
+      const float* src = row + v_col0 + (size_t)head * Dv;
+      const float* b = bias_v ? bias_v + (size_t)head * Dv : nullptr;
+      for (int u = lane; u < vhalf; u += 32) {
+        const int i0 = interleaved ? 2 * u : u, i1 = interleaved ? 2 * u + 1 : u + vhalf;
+        const float x0 = src[i0] + (b ? b[i0] : 0.f), x1 = src[i1] + (b ? b[i1] : 0.f);
+        const float sn = vsn_s[u], cs = vcs_s[u];
+        dst[i0] = from_float<T>(x0 * cs - x1 * sn);
+        dst[i1] = from_float<T>(x1 * cs + x0 * sn);
       }
+      for (int d = 2 * vhalf + lane; d < Dv; d += 32) dst[d] = from_float<T>(src[d] + (b ? b[d] : 0.f));
+      if (!rows_layout)
+        for (int d = Dv + lane; d < P; d += 32) dst[d] = from_float<T>(0.f);
+    }
+  }
+}
+
+// In place: every head of o [T, H * P] has its first Dv dimensions turned by -pos * freq[m] (pairs (m, m + Dv/2), or
+// (2m, 2m + 1) interleaved): what attention over turned values leaves is turned back by the row's own position.
+// VEC: four pairs a thread, 16- or 8-byte accesses.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+turn_back_kernel(T* __restrict__ o, const int* __restrict__ positions, const float* __restrict__ freq, int H, int Dv,
+                 int P, int interleaved) {
+  extern __shared__ __align__(16) float cs_s[];       // [Dv / 2] cosines, [Dv / 2] sines
+  const int t = blockIdx.x, half = Dv / 2;
+  float* sn_s = cs_s + half;
+  chain_release_if_small();
+  const int pos = positions[t];                       // a step's input, not the kernel before's output
+  for (int u = threadIdx.x; u < half; u += blockDim.x) {
+    float sn, cs;
+    sincosf((float)pos * freq[u], &sn, &cs);
+    cs_s[u] = cs;
+    sn_s[u] = sn;
+  }
+  __syncthreads();
+  chain_wait(o);
+  T* row = o + (size_t)t * H * P;
+  if constexpr (VEC) {
+    const int q = half / 4;
+    for (int i = threadIdx.x; i < H * q; i += blockDim.x) {
+      const int hd = i / q, m = (i - hd * q) * 4;
+      T* p = row + (size_t)hd * P;
+      T* p0 = interleaved ? p + 2 * m : p + m;
+      T* p1 = interleaved ? p + 2 * m + 4 : p + m + half;
+      float x[4], z[4], a[4], b[4];
+      load4(p0, x);
+      load4(p1, z);
+      // interleaved: x = (a0 b0 a1 b1), z = (a2 b2 a3 b3)
+      const float u0[4] = {x[0], interleaved ? x[2] : x[1], interleaved ? z[0] : x[2], interleaved ? z[2] : x[3]};
+      const float u1[4] = {interleaved ? x[1] : z[0], interleaved ? x[3] : z[1], interleaved ? z[1] : z[2], z[3]};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        a[e] = u0[e] * cs_s[m + e] + u1[e] * sn_s[m + e];
+        b[e] = u1[e] * cs_s[m + e] - u0[e] * sn_s[m + e];
+      }
+      const float w0[4] = {a[0], interleaved ? b[0] : a[1], interleaved ? a[1] : a[2], interleaved ? b[1] : a[3]};
+      const float w1[4] = {interleaved ? a[2] : b[0], interleaved ? b[2] : b[1], interleaved ? a[3] : b[2], b[3]};
+      store4(p0, w0);
+      store4(p1, w1);
+    }
+  } else {
+    for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
+      const int hd = i / half, m = i - hd * half;
+      T* p = row + (size_t)hd * P;
+      const int i0 = interleaved ? 2 * m : m, i1 = interleaved ? 2 * m + 1 : m + half;
+      const float a = to_float(p[i0]), b = to_float(p[i1]);
+      p[i0] = from_float<T>(a * cs_s[m] + b * sn_s[m]);
+      p[i1] = from_float<T>(b * cs_s[m] - a * sn_s[m]);
+    }
   }
 }
 
@@ -227,32 +314,55 @@ extern "C" int nf_qk_whole_norm_append(const float* proj, int ld, int q_col0, in
 }
 
 // proj float32 [T, ld]: q (Hq x D) at q_col0, and with Hkv > 0 k (Hkv x D) at k_col0 and v (Hkv x Dv) at
-// v_col0.  rows_layout 0: pages [.., 2, Hkv, page_size, D] (Dv == D); 1: pages [.., page_size, Hkv * (D + Dv)].
+// v_col0.  rows_layout 0: pages [.., 2, Hkv, page_size, P], P >= max(D, Dv); 1: pages [.., page_size, Hkv * (D + Dv)].
+// q_out [T, Hq * P].  wq (and wk) null: no norms.  v_freq float32 [Dv / 2] or null: values turned.
 extern "C" int nf_whole_norm_rope_append(const float* proj, int ld, int q_col0, int k_col0, int v_col0,
                                          const float* bias_q, const float* bias_k, const float* bias_v,
                                          const float* wq, const float* wk, float eps, const float* inv_freq, int rot,
                                          float mag, const int* positions, const int* row_seg, void* q_out, int T,
                                          int Hq, int Hkv, int D, int Dv, void* pages, const int* block_table,
-                                         int bt_width, int page_size, int num_pages, int rows_layout, int dtype,
-                                         cudaStream_t stream) {
+                                         int bt_width, int page_size, int num_pages, int rows_layout, int P,
+                                         int interleaved, const float* v_freq, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
-  NF_REQUIRE(T > 0 && Hq > 0 && Hkv >= 0 && D > 0 && Dv > 0 && wq && (Hkv == 0 || wk), "whole_norm_rope_append: bad arguments");
+  NF_REQUIRE(T > 0 && Hq > 0 && Hkv >= 0 && D > 0 && Dv > 0 && (!wq || Hkv == 0 || wk), "whole_norm_rope_append: bad arguments");
   NF_REQUIRE(q_col0 >= 0 && q_col0 + Hq * D <= ld, "whole_norm_rope_append: the queries leave the projection");
   NF_REQUIRE(Hkv == 0 || (k_col0 >= 0 && v_col0 >= 0 && k_col0 + Hkv * D <= ld && v_col0 + Hkv * Dv <= ld),
              "whole_norm_rope_append: keys or values leave the projection");
   NF_REQUIRE(Hkv == 0 || (pages && block_table), "whole_norm_rope_append: keys without a cache");
   NF_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= D && (rot == 0 || inv_freq), "whole_norm_rope_append: %d turned dimensions of %d", rot, D);
-  NF_REQUIRE(rows_layout || Hkv == 0 || D == Dv, "whole_norm_rope_append: the head-major page needs equal key and value sizes");
-  const size_t smem = ((size_t)(Hq + Hkv) * D + rot) * sizeof(float);
+  NF_REQUIRE(P >= D && (rows_layout || Hkv == 0 || P >= Dv), "whole_norm_rope_append: heads of %d and %d do not fit rows of %d", D, Dv, P);
+  NF_REQUIRE(!v_freq || Dv % 2 == 0, "whole_norm_rope_append: values of %d cannot be turned in pairs", Dv);
+  const size_t smem = ((size_t)(Hq + Hkv) * D + rot + (v_freq ? Dv : 0)) * sizeof(float);
   NF_REQUIRE(smem <= 200 * 1024, "whole_norm_rope_append: %d values a row do not fit shared memory", (Hq + Hkv) * D);
   if (dtype == kF32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(whole_norm_rope_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_chained(whole_norm_rope_append_kernel<float>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (float*)q_out, Hq, Hkv, D, Dv, (float*)pages, block_table, bt_width, page_size, num_pages, rows_layout);
+    launch_chained(whole_norm_rope_append_kernel<float>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (float*)q_out, Hq, Hkv, D, Dv, (float*)pages, block_table, bt_width, page_size, num_pages, rows_layout, P, interleaved, v_freq);
   } else {
     if (smem > 48 * 1024) cudaFuncSetAttribute(whole_norm_rope_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_chained(whole_norm_rope_append_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (__nv_bfloat16*)q_out, Hq, Hkv, D, Dv, (__nv_bfloat16*)pages, block_table, bt_width, page_size, num_pages, rows_layout);
+    launch_chained(whole_norm_rope_append_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (__nv_bfloat16*)q_out, Hq, Hkv, D, Dv, (__nv_bfloat16*)pages, block_table, bt_width, page_size, num_pages, rows_layout, P, interleaved, v_freq);
   }
   return check_launch("whole_norm_rope_append");
+}
+
+// o [T, H * P] of `dtype`, in place; freq float32 [Dv / 2].
+extern "C" int nf_turn_back(void* o, const int* positions, const float* freq, int T, int H, int Dv, int P,
+                            int interleaved, int dtype, cudaStream_t stream) {
+  if (T == 0) return 0;
+  NF_REQUIRE(T > 0 && H > 0 && Dv > 0 && Dv % 2 == 0 && P >= Dv && Dv <= 8192, "turn_back: bad sizes H=%d Dv=%d P=%d", H, Dv, P);
+  const size_t el = dtype == kF32 ? 4 : 2;
+  const bool vec = Dv % 8 == 0 && P % 4 == 0 && (uintptr_t)o % (4 * el) == 0;
+  const size_t smem = (size_t)Dv * sizeof(float);
+  const int units = vec ? H * Dv / 8 : H * Dv / 2;
+  int th = 32;
+  while (th < units && th < 256) th <<= 1;
+  if (dtype == kF32) {
+    if (vec) launch_chained(turn_back_kernel<float, true>, dim3(T), dim3(th), smem, stream, (float*)o, positions, freq, H, Dv, P, interleaved);
+    else launch_chained(turn_back_kernel<float, false>, dim3(T), dim3(th), smem, stream, (float*)o, positions, freq, H, Dv, P, interleaved);
+  } else {
+    if (vec) launch_chained(turn_back_kernel<__nv_bfloat16, true>, dim3(T), dim3(th), smem, stream, (__nv_bfloat16*)o, positions, freq, H, Dv, P, interleaved);
+    else launch_chained(turn_back_kernel<__nv_bfloat16, false>, dim3(T), dim3(th), smem, stream, (__nv_bfloat16*)o, positions, freq, H, Dv, P, interleaved);
+  }
+  return check_launch("turn_back");
 }
 
 // o, out [T, width] of `dtype`; g [T, ldg] float32 (g_dtype 0) or of `dtype`.

@@ -334,13 +334,14 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ X, int ldx, const __nv_bflo
       if (f < N) Y[(size_t)row * ldy + f] = from_float<TC>(gated_act(lo, hi, act));
     } else {
       const int f0 = n0 + gg, f1 = n0 + gg + 8;
+      if (act.kind == kActRelu2) { lo = relu_square(lo); hi = relu_square(hi); }
       if (f0 < N) Y[(size_t)row * ldy + f0] = from_float<TC>(lo);
       if (f1 < N) Y[(size_t)row * ldy + f1] = from_float<TC>(hi);
     }
   }
 }
 
-static thread_local GatedActParams t_gated_act{kActSilu, 0.f, 0.f};   // the current call's gated epilogue
+static thread_local GatedActParams t_gated_act{kActNone, 0.f, 0.f};   // the current call's epilogue
 
 int g_skinny_max_split = kMaxSplit;      // nf_set_skinny_max_split(): 1 turns the split over k off
 
@@ -391,7 +392,8 @@ using namespace nf;
 // Y[M, N] = epilogue(X[M, K] W[g]^T), bfloat16 inputs, float32 accumulation.
 // out_dtype: 1 bfloat16, 0 float32.  max_rows: bound on the rows of any one group.
 // Needs K % 8 == 0 and 16-byte aligned rows (ldx % 8 == 0, bases aligned).
-// swiglu: 0 none, 1 silu(gate) * up, 2 the capped form of common.cuh (act_limit, act_alpha).
+// swiglu: 0 none, 1 silu(gate) * up, 2 the capped form of common.cuh (act_limit, act_alpha), 4 gelu_tanh(gate) * up;
+// 5: no gate, the square of relu of each sum (W has N rows).
 // packed != 0: W is in the packed tile layout (w_group_stride then counts packed elements).
 // group_map / n_mapped: optional list of the groups to run (-1 entries are skipped); the grid
 // then has n_mapped groups instead of `groups`.  early_index != 0: offsets, x_rows and group_map
@@ -412,10 +414,10 @@ extern "C" int nf_skinny_gemm(const void* X, int ldx, const void* W, long long w
   // next to each other so that the second reading comes from L2
   const int nt = max_rows <= 8 ? 1 : 2;
   const size_t wgs = (size_t)w_group_stride;
-  if (swiglu) {
+  t_gated_act = GatedActParams{swiglu, act_limit, act_alpha};
+  if (swiglu && swiglu != kActRelu2) {
     NF_REQUIRE(out_dtype == kBF16, "skinny_gemm: the SwiGLU epilogue writes bfloat16");
     NF_REQUIRE(swiglu == kActSilu || swiglu == kActCapped || swiglu == kActGeluTanh, "skinny_gemm: gated epilogue %d", swiglu);
-    t_gated_act = GatedActParams{swiglu, act_limit, act_alpha};
     return launch_sw<true, __nv_bfloat16>(nt, packed != 0, X, ldx, W, wgs, Y, ldy, M, N, K, groups, max_rows, offsets, x_rows, x_div, group_map, n_mapped, early_index, stream);
   }
   if (out_dtype == kBF16)

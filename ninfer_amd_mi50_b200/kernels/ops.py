@@ -143,13 +143,14 @@ def capped_activation(limit: float, alpha: float) -> Tuple[int, float, float]:
     return (2, float(limit), float(alpha))
 
 
+ACT_RELU2 = (5, 0.0, 0.0)         # no gate: the square of relu of a product's sums
 ACT_GELU_TANH = (4, 0.0, 0.0)     # gelu_tanh(gate) * up, gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 
 
 def _act(swiglu, act) -> Tuple[int, float, float]:
-    """The epilogue a product is launched with: none, or the gated activation `act`."""
+    """The epilogue a product is launched with: none, the gated activation `act`, or one without a gate."""
     if not swiglu:
-        return (0, 0.0, 0.0)
+        return ACT_RELU2 if act == ACT_RELU2 else (0, 0.0, 0.0)
     return ACT_SILU if act is None else act
 
 
@@ -181,11 +182,11 @@ def _chk(t: torch.Tensor, name: str, dtype=None, contiguous=True) -> None:
 # rows
 # ---------------------------------------------------------------------------------------
 
-def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t] = float32(table[ids[t]])."""
+def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t] = float32(table[ids[t]]) * scale."""
     _chk(table, "table"); _chk(ids, "ids", torch.int32); _chk(out, "out", torch.float32)
     _lib.call("nf_embed_rows", _p(table), _p(ids), _p(out), c_int(ids.numel()),
-              c_int(table.shape[1]), c_int(table.shape[0]), c_int(_dt(table)), _stream())
+              c_int(table.shape[1]), c_int(table.shape[0]), c_float(scale), c_int(_dt(table)), _stream())
 
 
 def add_rmsnorm(h: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
@@ -207,6 +208,20 @@ def add_rmsnorm_rows(h: torch.Tensor, delta: Optional[torch.Tensor], rows: torch
         _chk(delta, "delta", out.dtype)
     _lib.call("nf_add_rmsnorm", _p(h), _p(delta), _p(rows), _p(weight), c_float(eps), _p(out),
               c_int(rows.numel()), c_int(h.shape[1]), c_int(_dt(out)), _stream())
+
+
+def add_group_rmsnorm(h: torch.Tensor, d1: Optional[torch.Tensor], d2: Optional[torch.Tensor], rows: Optional[torch.Tensor],
+                      weight: torch.Tensor, eps: float, groups: int, out: torch.Tensor) -> None:
+    """h += d1 (+ d2) (float32, in place); out = each of `groups` equal parts of h over its own root mean
+    square, times weight.  With `rows`: out[r] from h[rows[r]] + d1[rows[r]] + d2[rows[r]], h left as it is."""
+    _chk(h, "h", torch.float32); _chk(weight, "weight", torch.float32); _chk(out, "out")
+    for d, n in ((d1, "d1"), (d2, "d2")):
+        if d is not None:
+            _chk(d, n, out.dtype)
+    if rows is not None:
+        _chk(rows, "rows", torch.int32)
+    _lib.call("nf_add_group_rmsnorm", _p(h), _p(d1), _p(d2), _p(rows), _p(weight), c_float(eps), c_int(groups), _p(out),
+              c_int(out.shape[0]), c_int(h.shape[1]), c_int(_dt(out)), _stream())
 
 
 def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
@@ -380,6 +395,26 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
     return out
 
 
+def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """relu(x w^T)^2, x [M, K], w [N, K] -> [M, N]: in the product's epilogue on its float32 sums, or as one
+    pass over the float32 sums of a library product."""
+    _chk(x, "x"); _chk(w, "w", x.dtype)
+    M, K = x.shape
+    N = w.shape[0]
+    out = torch.empty((M, N), dtype=x.dtype, device=x.device)
+    if M == 0:
+        return out
+    path = "simt" if x.dtype == torch.float32 else _bf16_path(M, K, "bf16_linear")
+    if path == "skinny":
+        _skinny(x, K, w, 0, out, M, N, K, 1, M, None, None, 1, False, act=ACT_RELU2)
+    elif path == "simt":
+        _gemm_simt(x, K, w, 0, out, M, N, K, 1, M, None, None, 1, False, act=ACT_RELU2)
+    else:
+        z = linear(x, w, out_dtype=torch.float32)
+        _lib.call("nf_relu_square", _p(z), _p(out), c_longlong(z.numel()), c_int(_dt(out)), _stream())
+    return out
+
+
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, act=None) -> torch.Tensor:
     """x [M, K], w [2I, K] (gate rows first) -> silu(x gate^T) * (x up^T)  [M, I]; `act`: another gated
     activation in silu's place (the product kernels' epilogues take it; after a library product it is a
@@ -537,7 +572,7 @@ def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.T
             _lib.call("nf_prefill_attention_tc", _p(qkv), c_longlong(T), c_int(qkv.shape[1]), _p(pages),
                       _p(block_table), c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0),
                       _p(tiles), c_int(n_tiles), _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
-                      c_int(pages.shape[0]), c_int(window), c_float(scale), _stream())
+                      c_int(pages.shape[0]), c_int(window), c_float(scale), None, _stream())
             return out
         tiles, n_tiles = _tiles(ctx, PREFILL_TILE_ROWS, window, PREFILL_KEY_BLOCK, True, min_rows)
         _lib.call("nf_prefill_attention", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
@@ -549,7 +584,7 @@ def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.T
               _p(block_table), c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg),
               _p(out), c_int(T), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
               c_int(pages.shape[0]), c_int(window), c_float(scale), c_int(_dt(qkv)), None, c_int(0), None,
-              c_int(0), _stream())
+              c_int(0), None, _stream())
     return out
 
 
@@ -579,31 +614,47 @@ def whole_norm_rope_append(proj: torch.Tensor, q_col0: int, k_col0: int, v_col0:
                            bias_k: Optional[torch.Tensor], bias_v: Optional[torch.Tensor], wq: torch.Tensor,
                            wk: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rot: int,
                            magnitude: float, Hq: int, Hkv: int, D: int, Dv: int, ctx, pages: Optional[torch.Tensor],
-                           block_table: Optional[torch.Tensor], page_size: int, out_dtype: torch.dtype) -> torch.Tensor:
+                           block_table: Optional[torch.Tensor], page_size: int, out_dtype: torch.dtype,
+                           interleaved: bool = False, value_freq: Optional[torch.Tensor] = None, row: int = 0) -> torch.Tensor:
     """proj float32 [T, ld] holds q (Hq x D) at q_col0 and, with Hkv > 0, k (Hkv x D) at k_col0 and v (Hkv x Dv)
     at v_col0.  Adds the biases; q and k each over the root mean square of their whole row slice, times wq / wk
     (of the slice's width); the first `rot` dimensions of every q and k head turned by the row's position (pairs
     (i, i + rot/2), inv_freq float32 [rot / 2]), cosine and sine times `magnitude`.  Returns q [T, Hq * D] in
     `out_dtype` and writes key and value at (request, position): into pages [n, 2, Hkv, page_size, D] (then
     Dv == D) or, when `pages` has three dimensions, into rows [n, page_size, Hkv * (D + Dv)].  Hkv = 0: the
-    queries alone."""
-    _chk(proj, "proj", torch.float32); _chk(wq, "wq", torch.float32)
-    for b, n in ((bias_q, "bias_q"), (bias_k, "bias_k"), (bias_v, "bias_v"), (wk, "wk"), (inv_freq, "inv_freq")):
+    queries alone.  wq None: no norms.  `interleaved`: pairs (2i, 2i + 1).  `value_freq` (float32 [Dv / 2]): the
+    values are turned as well, over all their dimensions in the same layout of pairs.  `row` > D: queries, keys and
+    values are widened with zeros to that many numbers a head (pages [n, 2, Hkv, page_size, row], q [T, Hq * row])."""
+    _chk(proj, "proj", torch.float32)
+    for b, n in ((bias_q, "bias_q"), (bias_k, "bias_k"), (bias_v, "bias_v"), (wq, "wq"), (wk, "wk"), (inv_freq, "inv_freq"),
+                 (value_freq, "value_freq")):
         if b is not None:
             _chk(b, n, torch.float32)
     T = proj.shape[0]
-    q = torch.empty((T, Hq * D), dtype=out_dtype, device=proj.device)
+    P = row or D
+    q = torch.empty((T, Hq * P), dtype=out_dtype, device=proj.device)
     rows_layout = 0
     if Hkv:
         _chk(pages, "pages", out_dtype); _chk(block_table, "block_table", torch.int32)
         rows_layout = 1 if pages.dim() == 3 else 0
+        if not rows_layout and pages.shape[-1] != P:
+            raise ValueError(f"whole_norm_rope_append: pages of {pages.shape[-1]} numbers a head, rows of {P}")
     _lib.call("nf_whole_norm_rope_append", _p(proj), c_int(proj.shape[1]), c_int(q_col0), c_int(k_col0), c_int(v_col0),
               _p(bias_q), _p(bias_k), _p(bias_v), _p(wq), _p(wk), c_float(eps), _p(inv_freq) if rot else None, c_int(rot),
               c_float(magnitude), _p(ctx.positions), _p(ctx.row_seg), _p(q), c_int(T), c_int(Hq), c_int(Hkv), c_int(D),
               c_int(Dv), _p(pages) if Hkv else None, _p(block_table) if Hkv else None,
               c_int(block_table.shape[1] if Hkv else 0), c_int(page_size), c_int(pages.shape[0] if Hkv else 0),
-              c_int(rows_layout), c_int(_dt(q)), _stream())
+              c_int(rows_layout), c_int(P), c_int(1 if interleaved else 0), _p(value_freq), c_int(_dt(q)), _stream())
     return q
+
+
+def turn_back(o: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, H: int, Dv: int, row: int = 0,
+              interleaved: bool = False) -> None:
+    """In place: the first Dv numbers of every head of o [T, H * (row or Dv)] turned by minus the row's position
+    (pair m by freq[m], float32 [Dv / 2]; pairs (m, m + Dv/2), or (2m, 2m + 1) interleaved)."""
+    _chk(o, "o"); _chk(positions, "positions", torch.int32); _chk(freq, "freq", torch.float32)
+    _lib.call("nf_turn_back", _p(o), _p(positions), _p(freq), c_int(o.shape[0]), c_int(H), c_int(Dv), c_int(row or Dv),
+              c_int(1 if interleaved else 0), c_int(_dt(o)), _stream())
 
 
 def sigmoid_gate_rows(o: torch.Tensor, g_src: torch.Tensor, g_col0: int) -> torch.Tensor:
@@ -620,16 +671,19 @@ def sigmoid_gate_rows(o: torch.Tensor, g_src: torch.Tensor, g_col0: int) -> torc
 def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.Tensor, block_table: torch.Tensor,
                             page_size: int, ctx, window: int, keep_first: int, scale: float,
                             slopes: Optional[torch.Tensor], gate: Optional[torch.Tensor] = None,
-                            gate_col0: int = 0) -> torch.Tensor:
+                            gate_col0: int = 0, sigmoid_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal softmax attention of q [T, Hq * D] over the paged keys and values -> [T, Hq * D], with
     slopes[h] * (i - j) taken off head h's score of key j (float32 [Hq] or None), a window (0: none) that
     keeps the request's first `keep_first` keys visible, and head h's output times
-    sigmoid(gate[t, gate_col0 + h]) (gate float32 [T, ld] or None)."""
+    sigmoid(gate[t, gate_col0 + h]) (gate float32 [T, ld] or None).  With `sigmoid_bias` (float32 [Hq], then no
+    slopes) a visible key weighs sigmoid(score + sigmoid_bias[h]) instead, not normalised over keys."""
     _chk(q, "q"); _chk(pages, "pages", q.dtype); _chk(block_table, "block_table", torch.int32)
     if slopes is not None:
         _chk(slopes, "slopes", torch.float32)
     if gate is not None:
         _chk(gate, "gate", torch.float32)
+    if sigmoid_bias is not None:
+        _chk(sigmoid_bias, "sigmoid_bias", torch.float32)
     T = q.shape[0]
     out = torch.empty((T, Hq * D), dtype=q.dtype, device=q.device)
     if T == 0:
@@ -651,11 +705,22 @@ def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: t
                           c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0), _p(tiles), c_int(n_tiles),
                           _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window),
                           c_float(scale), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), c_int(shares), _p(part_o),
-                          _p(part_ml), _stream())
+                          _p(part_ml), _p(sigmoid_bias), _stream())
             singles, n_single = ctx.one_row_tiles()
             if n_single:
                 flash(singles, n_single, int(_lib.load().nf_prefill_attention_shares(c_int(window), c_int(int(ctx.max_context)))))
-            if not ctx.all_single:
+            if not ctx.all_single and (
+                    sigmoid_bias is not None and gate is None and T >= TUNING["prefill_attention_tc_min_rows"]
+                    and _lib.load().nf_prefill_attention_tc_fits(c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
+                                                                c_longlong(pages.shape[0]))):
+                # tcgen05 / TMEM / TMA: tiles of 128 rows, blocks of 128 keys
+                tiles, n_tiles = _tiles(ctx, 128, window, 128, False, 2 if n_single else 1)
+                if n_tiles:
+                    _lib.call("nf_prefill_attention_tc", _p(q), c_longlong(T), c_int(q.shape[1]), _p(pages), _p(block_table),
+                              c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0), _p(tiles), c_int(n_tiles),
+                              _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window),
+                              c_float(scale), _p(sigmoid_bias), _stream())
+            elif not ctx.all_single:
                 tiles, n_tiles = _tiles(ctx, PREFILL_TILE_ROWS, window, PREFILL_KEY_BLOCK, True, 2 if n_single else 1)
                 if n_tiles:
                     flash(tiles, n_tiles, 0)
@@ -663,7 +728,7 @@ def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: t
     _lib.call("nf_paged_attention_generic", _p(q), c_int(q.shape[1]), _p(pages), _p(block_table),
               c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg), _p(out), c_int(T), c_int(Hq),
               c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window), c_float(scale),
-              c_int(_dt(q)), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), _stream())
+              c_int(_dt(q)), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), _p(sigmoid_bias), _stream())
     return out
 
 
@@ -1213,13 +1278,14 @@ def add_row_vector(h: torch.Tensor, vec: torch.Tensor) -> None:
     _lib.call("nf_add_row_vector", _p(h), _p(vec), c_int(h.shape[0]), c_int(h.shape[1]), _stream())
 
 
-def heads_sigmoid_gate(v: torch.Tensor, g_src: torch.Tensor, g_col0: int) -> torch.Tensor:
-    """v [heads, T, n] (head-major) times sigmoid(g_src[:, g_col0 + head * n + i]) -> [T, heads * n]."""
+def heads_sigmoid_gate(v: torch.Tensor, g_src: torch.Tensor, g_col0: int, per_head: bool = False) -> torch.Tensor:
+    """v [heads, T, n] (head-major) times sigmoid(g_src[:, g_col0 + head * n + i]) -> [T, heads * n]; `per_head`: the
+    gate has one number a head, g_src[:, g_col0 + head]."""
     _chk(v, "v"); _chk(g_src, "g_src", v.dtype)
     heads, T, n = v.shape
     out = torch.empty((T, heads * n), dtype=v.dtype, device=v.device)
     _lib.call("nf_heads_sigmoid_gate", _p(v), _p(g_src), c_int(g_src.shape[1]), c_int(g_col0), _p(out), c_int(T),
-              c_int(heads), c_int(n), c_int(_dt(v)), _stream())
+              c_int(heads), c_int(n), c_int(1 if per_head else 0), c_int(_dt(v)), _stream())
     return out
 
 
@@ -1494,6 +1560,8 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, head_stride: int, rot
     head * head_stride + rot_off.  Returns [heads, T, R]."""
     _chk(q_abs, "q_abs"); _chk(q, "q", q_abs.dtype); _chk(pages, "pages", q_abs.dtype)
     heads, T, R = q_abs.shape
+    if Dr == 0:                             # no rotated part: the queries are q_abs alone, nothing else is read
+        q, head_stride, rot_off = q_abs.view(heads * T, R), R, 0
     if sink is not None:
         _chk(sink, "sink", torch.float32)
     out = torch.empty((heads, T, R), dtype=q_abs.dtype, device=q_abs.device)

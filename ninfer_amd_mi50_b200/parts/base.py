@@ -367,8 +367,18 @@ class StreamUpdate:
     out: Optional[torch.Tensor]
 
 
+@dataclass
+class PairSum:
+    """The outputs of a mixer and a feed-forward that ran side by side on one input, both still to be added
+    to the stream.  A norm that knows the form (`takes_pair`) adds both in its own pass, in 32-bit."""
+    a: torch.Tensor
+    b: torch.Tensor
+
+
 def summed(delta):
     """`delta` as a tensor (None stays None; a `StreamCopy` means nothing is left to add)."""
+    if isinstance(delta, PairSum):
+        return (delta.a.to(torch.float32) + delta.b.to(torch.float32)).to(delta.a.dtype)
     if isinstance(delta, StreamCopy):
         return None
     if isinstance(delta, BiasedOutput):
@@ -409,6 +419,12 @@ class PositionEncoding(Part):
         rotate-and-append kernel (half-split pairing), or None if the encoding is not of
         that form; then `apply` is called and the kernel appends without rotating."""
         return None
+
+    def pair_table(self, device: torch.device) -> Optional[Tuple[torch.Tensor, int, bool]]:
+        """(inverse frequencies float32 [rotary_dim // 2], rotary_dim, interleaved) for kernels that take
+        either layout of pairs: (i, i + rotary_dim / 2), or (2i, 2i + 1) interleaved."""
+        table = self.rotary_table(device)
+        return None if table is None else (*table, False)
 
     # what multiplies cosine and sine of every angle (a kernel that rotates takes it with the table)
     magnitude = 1.0

@@ -58,6 +58,79 @@ class PreNormBlock(Block):
         return self.feed_forward.forward(x2, ctx)
 
 
+@register_part("block", "parallel")
+class ParallelBlock(Block):
+    """One norm whose output both sublayers read, side by side: ``h += mixer(norm1(h)) + feed_forward(norm1(h))``.
+    Both outputs are left pending (`PairSum`), so that the next norm adds them to the stream in its own
+    pass.  In small steps, whose kernels do not fill the device, the feed-forward runs beside the mixer on a
+    second stream (a parallel branch of a captured graph).  A layer whose feed-forward is ``"none"`` is
+    ``h += mixer(norm1(h))``."""
+
+    # steps of up to this many rows run the feed-forward on the second stream; 0: never
+    fork_max_rows = 64
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm, feed_forward: FeedForward):
+        self.norm1, self.mixer, self.feed_forward = norm1, mixer, feed_forward      # (there is no second norm)
+
+    @property
+    def has_ff(self) -> bool:
+        return not getattr(self.feed_forward, "absent", False)
+
+    def parts(self):
+        return (self.norm1, self.mixer, self.feed_forward) if self.has_ff else (self.norm1, self.mixer)
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(p.graph_safe for p in self.parts())
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [s for p in self.parts() for s in p.tensor_specs()]
+
+    def load(self, fetch: Fetch) -> None:
+        for p in self.parts():
+            p.load(fetch)
+
+    def weight_bytes(self) -> int:
+        return sum(p.weight_bytes() for p in self.parts())
+
+    def check_limits(self, dtype, max_context, page_size) -> None:
+        for p in self.parts():
+            p.check_limits(dtype, max_context, page_size)
+
+    def settle(self, h: torch.Tensor, pending):
+        from .base import PairSum
+        if isinstance(pending, PairSum):
+            h.add_(pending.a.to(torch.float32)).add_(pending.b.to(torch.float32))
+            return None
+        return super().settle(h, pending)
+
+    def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache: Optional[CacheView],
+                state: Optional[torch.Tensor]):
+        from .. import kernels
+        from .base import PairSum
+        from .feedforward import _side_stream
+        if isinstance(pending, PairSum):
+            if not getattr(self.norm1, "takes_pair", False):
+                pending = summed(pending)
+        elif not self.norm1.takes_unsummed or not isinstance(pending, (torch.Tensor, RoutedSum, type(None))):
+            pending = summed(pending)
+        x = self.norm1.add_norm(h, pending, ctx.dtype)
+        if not self.has_ff:
+            return self.mixer.forward(x, ctx, cache, state)
+        if not (x.is_cuda and x.shape[0] <= self.fork_max_rows):
+            a = self.mixer.forward(x, ctx, cache, state)
+            return PairSum(a, summed(self.feed_forward.forward(x, ctx)))
+        main, side = torch.cuda.current_stream(x.device), _side_stream(x.device)
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            kernels.chain_break()               # its input comes from the other stream
+            f = summed(self.feed_forward.forward(x, ctx))
+        a = self.mixer.forward(x, ctx, cache, state)
+        main.wait_stream(side)
+        kernels.chain_break()                   # the kernel that adds both up also reads what the other stream produced
+        return PairSum(a, f)
+
+
 @register_part("block", "sublayer_norm_scaled")
 class SublayerNormScaledBlock(Block):
     """The norm sits on each sublayer's output, and a learned vector scales it per channel:

@@ -390,6 +390,38 @@ class SparseMoeSwiglu(FeedForward):
         return RoutedSum(y, plan, wts, shared, gate, x.dtype)
 
 
+@register_part("feed_forward", "dense_relu2")
+class DenseSquaredRelu(FeedForward):
+    """An ungated dense feed-forward ``W_down relu(W_up x)^2``.  The square is taken of the first product's
+    float32 sums: in its epilogue (few rows, and 32-bit mode), or in one pass over them after a library
+    product (many rows)."""
+
+    graph_safe = True
+    DEFAULT_NAMES = (("up", "up"), ("down", "down"))
+
+    def __init__(self, hidden_size: int, intermediate_size: int, prefix: str, tensor_names=None):
+        self.hidden_size, self.intermediate_size, self.prefix = int(hidden_size), int(intermediate_size), prefix
+        self.names = dict(self.DEFAULT_NAMES)
+        self.names.update(dict(tensor_names or ()))
+        self.w_up = self.w_down = None
+
+    def _n(self, what: str) -> str:
+        return self.prefix + self.names[what]
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        H, I = self.hidden_size, self.intermediate_size
+        return [TensorSpec(self._n("up"), (I, H)), TensorSpec(self._n("down"), (H, I))]
+
+    def load(self, fetch: Fetch) -> None:
+        self.w_up, self.w_down = fetch(self._n("up")), fetch(self._n("down"))
+
+    def weight_bytes(self) -> int:
+        return (self.w_up.numel() + self.w_down.numel()) * self.w_down.element_size()
+
+    def forward(self, x: torch.Tensor, ctx: StepContext):
+        return kernels.linear(kernels.linear_relu2(x, self.w_up), self.w_down)
+
+
 @register_part("feed_forward", "dense_poly_norm")
 class DensePolyNorm(FeedForward):
     """An ungated dense feed-forward ``W_down act(W_up x)`` whose activation is a polynomial of normed

@@ -17,7 +17,7 @@ import torch
 from .. import kernels
 from ..config.model_config import LayerCall, ModelPlan
 from ..registry import build_part, part_class
-from .base import CacheSpec, CacheView, Fetch, RoutedSum, StateSpec, StepContext, StreamUpdate, TensorSpec, summed
+from .base import CacheSpec, CacheView, Fetch, PairSum, RoutedSum, StateSpec, StepContext, StreamUpdate, TensorSpec, summed
 
 
 class DecoderModel:
@@ -40,6 +40,8 @@ class DecoderModel:
         self.streams = int(plan.streams)
         if not 1 <= self.streams <= kernels.MAX_STREAMS:
             raise ValueError(f"{self.streams} residual streams a token; the kernels take 1 to {kernels.MAX_STREAMS}")
+        if self.streams > 1 and plan.embedding_scale != 1.0:
+            raise ValueError("a scaled embedding and several residual streams do not go together")
         if self.streams > 1 and plan.embedding_extras:
             raise ValueError("rows added to the embedding and several residual streams do not go together")
         self.order: List[LayerCall] = list(plan.order)
@@ -135,7 +137,7 @@ class DecoderModel:
         """Run every row of the step; return float32 logits [R, vocab] for ctx.logit_rows."""
         h = torch.empty((ctx.T, self.hidden_size * self.streams), dtype=torch.float32, device=ctx.device)
         if self.streams == 1:
-            kernels.embed_rows(self.embedding, ctx.token_ids, h)
+            kernels.embed_rows(self.embedding, ctx.token_ids, h, scale=self.plan.embedding_scale)
         else:
             kernels.embed_copies(self.embedding, ctx.token_ids, h, self.streams)
         for i, e in enumerate(self.embedding_extras):
@@ -155,6 +157,8 @@ class DecoderModel:
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=ctx.device)
         if isinstance(pending, StreamUpdate) and getattr(self.final_norm, "takes_stream_update", False):
             pass                                     # the norm applies the update in its own pass over the rows
+        elif isinstance(pending, PairSum) and getattr(self.final_norm, "takes_pair", False):
+            pass                                     # ... and adds two contributions in it
         elif not self.final_norm.takes_unsummed or not isinstance(pending, (torch.Tensor, RoutedSum, type(None))):
             pending = summed(pending)
         x = self.final_norm.add_norm_rows(h, pending, ctx.logit_rows, ctx.dtype)

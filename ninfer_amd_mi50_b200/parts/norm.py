@@ -15,7 +15,7 @@ import torch
 
 from .. import kernels
 from ..registry import register_part
-from .base import Fetch, Norm, RoutedSum, TensorSpec, summed
+from .base import Fetch, Norm, PairSum, RoutedSum, TensorSpec, summed
 
 
 @register_part("norm", "rms_norm")
@@ -138,6 +138,7 @@ class GroupRmsNorm(Norm):
     graph_safe = True
     takes_unsummed = False
     takes_stream_update = True
+    takes_pair = True
 
     def __init__(self, size: int, eps: float, prefix: str, groups: int = 1, weight_name: str = "weight"):
         self.size, self.eps, self.prefix = int(size), float(eps), prefix
@@ -161,6 +162,12 @@ class GroupRmsNorm(Norm):
     def _apply(self, h, delta, rows, out_dtype):
         from .base import StreamUpdate
         S = h.shape[1] // self.size
+        if S == 1 and (delta is None or isinstance(delta, (torch.Tensor, PairSum))):
+            # the ordinary residual sum of one stream (of two contributions, if a mixer and a feed-forward ran side by side)
+            a, b = (delta.a, delta.b) if isinstance(delta, PairSum) else (delta, None)
+            out = torch.empty((h.shape[0] if rows is None else rows.numel(), self.size), dtype=out_dtype, device=h.device)
+            kernels.add_group_rmsnorm(h, a, b, rows, self.weight, self.eps, self.groups, out)
+            return out
         if isinstance(delta, StreamUpdate):
             y, mix, out = delta.y, delta.mix, delta.out
         else:

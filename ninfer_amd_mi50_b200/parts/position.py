@@ -29,10 +29,37 @@ def rotary_inverse_frequencies(head_dim: int, theta: float, rotary_dim: Optional
     return torch.from_numpy(inv)
 
 
+def double_inverse_frequencies(rotary_dim: int, theta: float) -> torch.Tensor:
+    """float32 [rotary_dim / 2]: theta^(-2i / rot), evaluated in double precision and rounded once."""
+    i = np.arange(int(rotary_dim) // 2, dtype=np.float64)
+    return torch.from_numpy(np.power(float(theta), -2.0 * i / int(rotary_dim)).astype(np.float32))
+
+
+def banded_inverse_frequencies(rotary_dim: int, theta: float, factor: float, low: float, high: float,
+                               original: float) -> torch.Tensor:
+    """float32 [rotary_dim / 2]: the plain frequencies f_i = theta^(-2i / rot) by bands of their wavelength
+    l = 2 pi / f (the Llama 3.1 rule): kept where l < original / high, divided by `factor` where
+    l > original / low, and between the two blended, (1 - s) f / factor + s f with
+    s = (original / l - low) / (high - low).  Evaluated in double precision, rounded once."""
+    import math
+    out = []
+    for i in range(int(rotary_dim) // 2):
+        f = float(theta) ** (-2.0 * i / int(rotary_dim))
+        wave = 2.0 * math.pi / f
+        if wave > original / low:
+            f = f / factor
+        elif wave >= original / high:
+            s = (original / wave - low) / (high - low) if high != low else 1.0
+            f = (1.0 - s) * f / factor + s * f
+        out.append(f)
+    return torch.tensor(out, dtype=torch.float64).to(torch.float32)
+
+
 @register_part("position", "rotary_half_split")
 class RotaryHalfSplit(PositionEncoding):
-    def __init__(self, head_dim: int, theta: float, rotary_dim: Optional[int] = None):
-        self.head_dim, self.theta = int(head_dim), float(theta)
+    def __init__(self, head_dim: int, theta: float, rotary_dim: Optional[int] = None, double: bool = False):
+        """`double`: the frequencies are evaluated in double precision and rounded once."""
+        self.head_dim, self.theta, self.double = int(head_dim), float(theta), bool(double)
         self.rotary_dim = int(head_dim if rotary_dim is None else rotary_dim)
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= self.head_dim:
             raise ValueError(f"rotary_dim={self.rotary_dim} must be even and in (0, {head_dim}]")
@@ -41,8 +68,9 @@ class RotaryHalfSplit(PositionEncoding):
     def rotary_table(self, device: torch.device) -> Optional[Tuple[torch.Tensor, int]]:
         key = str(device)
         if key not in self._table:
-            self._table[key] = rotary_inverse_frequencies(
-                self.head_dim, self.theta, self.rotary_dim).to(device)
+            table = (double_inverse_frequencies(self.rotary_dim, self.theta) if self.double
+                     else rotary_inverse_frequencies(self.head_dim, self.theta, self.rotary_dim))
+            self._table[key] = table.to(device)
         return self._table[key], self.rotary_dim
 
 
@@ -89,6 +117,45 @@ class RotaryHalfSplitBlended(RotaryHalfSplit):
             self._table[key] = blended_inverse_frequencies(self.rotary_dim, self.theta, self.factor, self.original,
                                                            self.fast, self.slow).to(device)
         return self._table[key], self.rotary_dim
+
+
+@register_part("position", "rotary_half_split_banded")
+class RotaryHalfSplitBanded(RotaryHalfSplit):
+    """The half-split rotation with frequencies scaled by bands of their wavelength
+    (`banded_inverse_frequencies`); cosine and sine are not scaled."""
+
+    def __init__(self, head_dim: int, theta: float, factor: float, low: float, high: float, original: float,
+                 rotary_dim: Optional[int] = None):
+        super().__init__(head_dim, theta, rotary_dim)
+        self.factor, self.low, self.high, self.original = float(factor), float(low), float(high), float(original)
+        if not (self.factor > 0 and self.low > 0 and self.high >= self.low and self.original > 0 and self.theta > 0):
+            raise ValueError("banded rotation: factor, original and base positive, 0 < low <= high")
+
+    def rotary_table(self, device: torch.device) -> Optional[Tuple[torch.Tensor, int]]:
+        key = str(device)
+        if key not in self._table:
+            self._table[key] = banded_inverse_frequencies(self.rotary_dim, self.theta, self.factor, self.low, self.high,
+                                                          self.original).to(device)
+        return self._table[key], self.rotary_dim
+
+
+@register_part("position", "rotary_interleaved")
+class RotaryInterleaved(PositionEncoding):
+    """The rotation whose pairs are neighbours: dimension 2i with 2i + 1, by pos * theta^(-2i / rot).  For
+    kernels that take a layout of pairs (`pair_table`); `rotary_table` promises half-split pairs and gives None."""
+
+    def __init__(self, head_dim: int, theta: float, rotary_dim: Optional[int] = None):
+        self.head_dim, self.theta = int(head_dim), float(theta)
+        self.rotary_dim = int(head_dim if rotary_dim is None else rotary_dim)
+        if self.rotary_dim % 2 or not 0 < self.rotary_dim <= self.head_dim:
+            raise ValueError(f"rotary_dim={self.rotary_dim} must be even and in (0, {head_dim}]")
+        self._table = {}
+
+    def pair_table(self, device: torch.device) -> Optional[Tuple[torch.Tensor, int, bool]]:
+        key = str(device)
+        if key not in self._table:
+            self._table[key] = double_inverse_frequencies(self.rotary_dim, self.theta).to(device)
+        return self._table[key], self.rotary_dim, True
 
 
 @register_part("position", "none")

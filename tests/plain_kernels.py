@@ -21,8 +21,8 @@ def _f(t):
     return t.to(torch.float32) if t.dtype in (torch.bfloat16, torch.float16) else t
 
 
-def embed_rows(table, ids, out):
-    out.copy_(_f(table)[ids.long()])
+def embed_rows(table, ids, out, scale=1.0):
+    out.copy_(_f(table)[ids.long()] * scale)
 
 
 def add_rmsnorm(h, delta, weight, eps, out):
