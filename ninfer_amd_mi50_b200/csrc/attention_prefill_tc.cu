@@ -502,11 +502,10 @@ extern "C" int nf_prefill_attention_tc_fits(int Hq, int Hkv, int D, int page_siz
 // every CTA two tiles as (segment, first row), each at most 128 consecutive rows of one segment;
 // the second may be (-1, -1).  qkv is [T, q_row_stride] with the queries in its first Hq * D
 // columns; out is [T, Hq * D].  sig_bias float32 [Hq] or null: sigmoid weights in the softmax's place.
-extern "C" int nf_prefill_attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages,
-                                       const int* block_table, int bt_width, const int* positions,
-                                       const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
-                                       int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                                       const float* sig_bias, cudaStream_t stream) {
+static int attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages, const int* block_table,
+                        int bt_width, const int* positions, const int* seg_row0, const int* tiles, int n_tiles,
+                        void* out, int Hq, int Hkv, int D, int page_size, int num_pages, int window, float scale,
+                        const float* sig_bias, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   NF_REQUIRE(n_tiles > 0 && n_tiles <= 65535 && T > 0, "prefill attention: bad sizes tiles=%d T=%lld", n_tiles, T);
   NF_REQUIRE(nf_prefill_attention_tc_fits(Hq, Hkv, D, page_size, num_pages), "prefill attention: sizes the tensor-core kernel does not take (Hq=%d Hkv=%d D=%d page=%d)", Hq, Hkv, D, page_size);
@@ -518,6 +517,25 @@ extern "C" int nf_prefill_attention_tc(const void* qkv, long long T, int q_row_s
   if (D == 64) return sig_bias ? NF_TC(64, true) : NF_TC(64, false);
   return sig_bias ? NF_TC(128, true) : NF_TC(128, false);
 #undef NF_TC
+}
+
+extern "C" int nf_prefill_attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages,
+                                       const int* block_table, int bt_width, const int* positions,
+                                       const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
+                                       int Hkv, int D, int page_size, int num_pages, int window, float scale,
+                                       cudaStream_t stream) {
+  return attention_tc(qkv, T, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq,
+                      Hkv, D, page_size, num_pages, window, scale, nullptr, stream);
+}
+
+extern "C" int nf_sigmoid_attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages,
+                                       const int* block_table, int bt_width, const int* positions,
+                                       const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
+                                       int Hkv, int D, int page_size, int num_pages, int window, float scale,
+                                       const float* sig_bias, cudaStream_t stream) {
+  NF_REQUIRE(sig_bias, "sigmoid attention needs its bias a head");
+  return attention_tc(qkv, T, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq,
+                      Hkv, D, page_size, num_pages, window, scale, sig_bias, stream);
 }
 
 // 0 if no tensor-core attention kernel has given up on a wait since the last call; else the code

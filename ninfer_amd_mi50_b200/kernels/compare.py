@@ -5,6 +5,7 @@ every kernel of one step timed by name against its roofline.
     python bench.py --config difavik
     python bench.py --config fetezen
     python bench.py --config kopadra
+    python bench.py --config pudizen
 
 For each named size a Vekasun model (latent attention and state-space mixers alternating, routed
 experts scored by a sigmoid and weighted on their input) and a Qwen2-MoE model of the same width,
@@ -108,6 +109,28 @@ def kopadra_config(s: dict) -> dict:
             "layers": [dict(m, mlp=f) for m, f in zip((att(None), att(0), rec, att(None)), mlps)]}
 
 
+# the Pudizen design at the same sizes: as many key heads as query heads, heads of 128 with half of them turned
+# (frequencies scaled by bands), a window of 1,024 keys for the sigmoid weights, a latent of the other comparisons'
+# size, a dense feed-forward of four times the width; the Qwen2-MoE model beside it has dense layers throughout, whose
+# three matrices hold as many weights as the design's two
+def pudizen_config(s: dict) -> dict:
+    H = s["heads"]
+    common = {"heads": H, "kv_heads": H, "dim": HEAD_DIM, "vdim": HEAD_DIM, "scale": HEAD_DIM ** -0.5}
+    att = {"type": "attention", "mixer": dict(common, rot={"base": 500000.0, "dims": ROT_DIM, "scaling": {
+        "factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}})}
+    win = {"type": "attention_2", "mixer": dict(common, rot={"base": 10000.0, "dims": ROT_DIM}, mask={"size": WINDOW})}
+    lat = {"type": "latent_attention", "mixer": {"heads": H, "dim": HEAD_DIM, "vdim": HEAD_DIM, "kv_rank": s["kv_rank"],
+                                                 "scale": HEAD_DIM ** -0.5}}
+    mlp = {"kind": "dense", "ff": 4 * s["width"]}
+    return {"architecture": "Pudizen", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6, "groups": NORM_GROUPS},
+            "embedding": {"scale": 8.0, "bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}},
+            "layers": [dict(m, mlp=mlp) for m in (att, win, lat, att)]}
+
+
+def qwen2_dense_config(s: dict) -> dict:
+    return dict(qwen2_moe_config(s), mlp_only_layers=list(range(LAYERS)), intermediate_size=4 * s["width"] * 2 // 3 // 64 * 64)
+
+
 def qwen2_moe_config(s: dict) -> dict:
     return {"architectures": ["Qwen2MoeForCausalLM"], "model_type": "qwen2_moe", "num_hidden_layers": LAYERS,
             "hidden_size": s["width"], "num_attention_heads": s["heads"], "num_key_value_heads": s["heads"],
@@ -178,6 +201,21 @@ def work_models(s: dict, prompt: int, batch: int, context: int, design: str = ""
                 "nf_identity_expert_rows": (T * k * W * 2 * 2 * IDENTITY / E, 0.0),
                 "nf_gated_bias_act": (T * k * s["ff"] * 2 * 3, 0.0),
             }
+        if design == "pudizen":
+            latent = (rows_ctx * R * 2 + 2 * T * H * R * 2, 4.0 * H * R * pairs)
+            own = {
+                "nf_latent_attention_mma": latent, "nf_latent_attention_generic": latent,
+                "nf_sigmoid_attention_tc": windowed,
+                # float32 sums of q, k, v in; q, key and value out
+                "nf_whole_norm_rope_append": (T * 3 * H * D * (4 + 2), 0.0),
+                "nf_turn_back": (T * H * D * (2 + 2), 0.0),
+                "nf_add_group_rmsnorm": (T * W * (8 + 2 + 2 + 2), 0.0),
+                "nf_relu_square": (T * 4 * W * (4 + 2), 0.0),
+                "nf_latent_append": (T * R * 4, 0.0),
+                "nf_silu_mul": (T * (4 * W * 2 // 3) * 2 * 3, 0.0),
+                "nf_heads_sigmoid_gate": (T * H * D * 4, 0.0),
+                "nf_embed_rows": (T * W * (2 + 4), 0.0),
+            }
         table = {
             # Fetezen: keys and values of the rows' chunks once, queries in and outputs out; both products and the
             # mixing of the heads' scores
@@ -221,7 +259,8 @@ def work_models(s: dict, prompt: int, batch: int, context: int, design: str = ""
         table.update(own)
         return table
 
-    seen = lambda p: min(p + 1, WINDOW) + max(0, min(KEEP_FIRST, p + 1 - WINDOW))       # keys position p sees
+    keep = 0 if design == "pudizen" else KEEP_FIRST
+    seen = lambda p: min(p + 1, WINDOW) + max(0, min(keep, p + 1 - WINDOW))             # keys position p sees
     in_chunk = lambda p: p % CHUNK + 1                                                  # keys position p sees in its chunk
     return {"prefill": phase(prompt, prompt * (prompt + 1) / 2, prompt, 1, float(sum(seen(p) for p in range(prompt))), prompt,
                              float(sum(in_chunk(p) for p in range(prompt))), prompt),
@@ -303,7 +342,9 @@ def measure(config: dict, prompt: int, batch: int, context: int, steps: int, war
     return out
 
 
-DESIGNS = {"vekasun": vekasun_config, "difavik": difavik_config, "fetezen": fetezen_config, "kopadra": kopadra_config}
+DESIGNS = {"vekasun": vekasun_config, "difavik": difavik_config, "fetezen": fetezen_config, "kopadra": kopadra_config,
+           "pudizen": pudizen_config}
+BESIDE = {"pudizen": qwen2_dense_config}            # the Qwen2-MoE model a design stands beside, where it is not the routed one
 
 
 def run_comparison(sizes, peaks: dict, prompt: int = 2048, batch: int = 8, context: int = 2048, steps: int = 32,
@@ -314,7 +355,7 @@ def run_comparison(sizes, peaks: dict, prompt: int = 2048, batch: int = 8, conte
         s = SIZES[name]
         models = work_models(s, prompt, batch, context, design)
         entry = {}
-        for which, cfg in ((design, DESIGNS[design](s)), ("qwen2_moe", qwen2_moe_config(s))):
+        for which, cfg in ((design, DESIGNS[design](s)), ("qwen2_moe", BESIDE.get(design, qwen2_moe_config)(s))):
             t0 = time.time()
             m = measure(cfg, prompt, batch, context, steps, warmup)
             for ph in ("prefill", "decode"):

@@ -572,7 +572,7 @@ def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.T
             _lib.call("nf_prefill_attention_tc", _p(qkv), c_longlong(T), c_int(qkv.shape[1]), _p(pages),
                       _p(block_table), c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0),
                       _p(tiles), c_int(n_tiles), _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
-                      c_int(pages.shape[0]), c_int(window), c_float(scale), None, _stream())
+                      c_int(pages.shape[0]), c_int(window), c_float(scale), _stream())
             return out
         tiles, n_tiles = _tiles(ctx, PREFILL_TILE_ROWS, window, PREFILL_KEY_BLOCK, True, min_rows)
         _lib.call("nf_prefill_attention", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
@@ -716,7 +716,7 @@ def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: t
                 # tcgen05 / TMEM / TMA: tiles of 128 rows, blocks of 128 keys
                 tiles, n_tiles = _tiles(ctx, 128, window, 128, False, 2 if n_single else 1)
                 if n_tiles:
-                    _lib.call("nf_prefill_attention_tc", _p(q), c_longlong(T), c_int(q.shape[1]), _p(pages), _p(block_table),
+                    _lib.call("nf_sigmoid_attention_tc", _p(q), c_longlong(T), c_int(q.shape[1]), _p(pages), _p(block_table),
                               c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0), _p(tiles), c_int(n_tiles),
                               _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window),
                               c_float(scale), _p(sigmoid_bias), _stream())
