@@ -12,6 +12,10 @@
 // order of every sum, depends on the row's own position (and window) only.
 //
 // All query heads of a group share the CTA, so keys and values are read once per kv head.
+//
+// Two further forms.  SIGMOID: a key weighs sigmoid(score + sig_bias[h]), not normalised over keys - blocks carry the
+// maximum 0 and simply add.  Turned values: the merge turns the first `turn_dims` numbers of a head's result by minus
+// the row's position (what turn_back in qk_norm_append.cu does in a pass of its own, here on the float32 sum).
 #define NF_CHAIN_CLASS 8
 #include "common.cuh"
 #include "decode_range.cuh"
@@ -60,7 +64,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 // weighted sum of values are tensor-core products with the keys (values) as the 16-row
 // operand and up to 8 query heads of the group as the 8-column operand; softmax stays in
 // float32 in between.  Warp w owns keys [32 w, 32 w + 32) of the block.
-template <int D>
+template <int D, bool SIGMOID>
 __global__ void __launch_bounds__(128)
 decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride,
                               const __nv_bfloat16* __restrict__ pages,
@@ -69,7 +73,7 @@ decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_s
                               float* __restrict__ ws_acc, float* __restrict__ ws_ml, int Hq, int Hkv,
                               int page_size, int num_pages, int window, float scale, int nsplit,
                               int* __restrict__ counters, __nv_bfloat16* __restrict__ out,
-                              const int* __restrict__ row_list) {
+                              const int* __restrict__ row_list, const float* __restrict__ sig_bias) {
   constexpr int LPR = D / 8;            // 16-byte pieces of one key row
   constexpr int RPL = 32 / LPR;         // key rows a warp copies at once
   constexpr int DS = D + 8;             // shared-memory row stride: 16 bytes of padding keep
@@ -201,6 +205,12 @@ decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_s
 
   // ---- per head: maximum, exponentials, sum (one warp per head) ----------------------------
   for (int h = warp; h < G; h += 4) {
+    if constexpr (SIGMOID) {
+      const float b = sig_bias[kvh * G + h];
+      for (int i = n0 + lane; i < n1; i += 32) sc[h * kSplit + i] = 1.f / (1.f + expf(-(sc[h * kSplit + i] + b)));
+      if (lane == 0) { ml[2 * h] = 0.f; ml[2 * h + 1] = 1.f; }
+      continue;
+    }
     float m = -INFINITY;
     for (int i = n0 + lane; i < n1; i += 32) m = fmaxf(m, sc[h * kSplit + i]);
     m = warp_max(m);
@@ -313,10 +323,12 @@ __global__ void decode_attention_merge_kernel(const float* __restrict__ ws_acc,
                                               const float* __restrict__ ws_ml,
                                               const int* __restrict__ positions, T* __restrict__ out,
                                               int Hq, int D, int window, int nsplit, int dthreads,
-                                              const int* __restrict__ row_list) {
+                                              const int* __restrict__ row_list, int normalise,
+                                              const float* __restrict__ turn_freq, int turn_dims, int interleaved) {
   extern __shared__ float runs[];      // [runs of this row][D]
   __shared__ float wgt[kMaxMergeSplits], wl[kMaxMergeSplits];
   __shared__ float s_m, s_inv;
+  __shared__ float fin[256];           // the head's result before it is turned
   const int wi = blockIdx.x, h = blockIdx.y;
   chain_release_if_small();
   // positions and the row list are the step's inputs, complete before the kernels of the step
@@ -348,7 +360,7 @@ __global__ void decode_attention_merge_kernel(const float* __restrict__ ws_acc,
   if (threadIdx.x == 0) {
     float l = 0.f;
     for (int s = 0; s < n; ++s) l += wl[s] * wgt[s];                              // ascending order
-    s_inv = l > 0.f ? 1.f / l : 0.f;
+    s_inv = !normalise ? 1.f : (l > 0.f ? 1.f / l : 0.f);
   }
   __syncthreads();
   // Runs of kMergeRun blocks are added by different thread groups (a long context has hundreds of
@@ -371,38 +383,58 @@ __global__ void decode_attention_merge_kernel(const float* __restrict__ ws_acc,
         o += a3 * wgt[s + 3];
       }
       for (; s < se; ++s) o += acc[(size_t)s * D + d] * wgt[s];
-      if (nruns == 1) out[((size_t)t * Hq + h) * D + d] = from_float<T>(o * s_inv);
-      else runs[(size_t)r * D + d] = o;
+      if (nruns > 1) runs[(size_t)r * D + d] = o;
+      else if (turn_freq) fin[d] = o * s_inv;
+      else out[((size_t)t * Hq + h) * D + d] = from_float<T>(o * s_inv);
     }
   }
-  if (nruns == 1) return;
+  if (nruns > 1) {
+    __syncthreads();
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+      float o = 0.f;
+      for (int r = 0; r < nruns; ++r) o += runs[(size_t)r * D + d];
+      if (turn_freq) fin[d] = o * s_inv;
+      else out[((size_t)t * Hq + h) * D + d] = from_float<T>(o * s_inv);
+    }
+  }
+  if (!turn_freq) return;
   __syncthreads();
+  const int half = turn_dims / 2;
+  const float p = (float)positions[t];
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    float o = 0.f;
-    for (int r = 0; r < nruns; ++r) o += runs[(size_t)r * D + d];
-    out[((size_t)t * Hq + h) * D + d] = from_float<T>(o * s_inv);
+    float v = fin[d];
+    if (d < turn_dims) {
+      const int m = interleaved ? d >> 1 : (d < half ? d : d - half);
+      const bool first = interleaved ? !(d & 1) : d < half;
+      const float other = fin[interleaved ? d ^ 1 : (first ? d + half : d - half)];
+      float sn, cs;
+      sincosf(p * turn_freq[m], &sn, &cs);
+      v = first ? v * cs + other * sn : v * cs - other * sn;
+    }
+    out[((size_t)t * Hq + h) * D + d] = from_float<T>(v);
   }
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 static int launch_split(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                         int bt_width, const int* positions, const int* row_seg, float* ws_acc,
                         float* ws_ml, int T, int Hq, int Hkv, int page_size, int num_pages, int window,
-                        float scale, int nsplit, int* counters, void* out, const int* row_list, cudaStream_t stream) {
+                        float scale, int nsplit, int* counters, void* out, const int* row_list, const float* sig_bias,
+                        cudaStream_t stream) {
   const int G = Hq / Hkv;
   const size_t smem = (size_t)2 * kSplit * (D + 8) * sizeof(__nv_bfloat16) +
                       ((size_t)G * kSplit + 4 * (G < 8 ? G : 8) * D + 2 * G) * sizeof(float);
   NF_REQUIRE(smem <= 200 * 1024, "decode attention: %d query heads per kv head need too much shared memory", G);
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
-    cudaFuncSetAttribute(decode_attention_split_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(decode_attention_split_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     allowed = smem;
   }
   dim3 grid(T, Hkv, nsplit);
-  launch_chained(decode_attention_split_kernel<D>, grid, dim3(128), smem, stream,
+  launch_chained(decode_attention_split_kernel<D, SIGMOID>, grid, dim3(128), smem, stream,
                  (const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width,
                  positions, row_seg, ws_acc, ws_ml, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters,
-                 (__nv_bfloat16*)out, row_list);
+                 (__nv_bfloat16*)out, row_list, sig_bias);
   return check_launch("decode_attention_split");
 }
 
@@ -414,7 +446,7 @@ int decode_attention_stream_fits(int T, int Hq, int Hkv, int D, int page_size);
 int decode_attention_stream(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                             int bt_width, const int* positions, const int* row_seg, float* ws_acc, float* ws_ml,
                             int T, int Hq, int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                            int nsplit, const int* row_list, cudaStream_t stream);
+                            int nsplit, const int* row_list, const float* sig_bias, cudaStream_t stream);
 int decode_attention_stream_status();
 int g_decode_stream = 1;
 }  // namespace nf
@@ -446,7 +478,8 @@ static int decode_attention_impl(const void* qkv, int q_row_stride, const void* 
                                  const int* row_seg, void* out, float* ws_acc, float* ws_ml, int T,
                                  int Hq, int Hkv, int D, int page_size, int num_pages, int window,
                                  float scale, int nsplit, int* counters, const int* row_list,
-                                 cudaStream_t stream) {
+                                 cudaStream_t stream, const float* sig_bias = nullptr,
+                                 const float* turn_freq = nullptr, int turn_dims = 0, int interleaved = 0) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0 && nsplit > 0, "decode attention: bad sizes T=%d Hq=%d Hkv=%d nsplit=%d", T, Hq, Hkv, nsplit);
   NF_REQUIRE(Hkv <= 65535 && nsplit <= kMaxMergeSplits, "decode attention: too many kv heads or key blocks (context beyond %d keys)", kMaxMergeSplits * kSplit);
@@ -456,18 +489,22 @@ static int decode_attention_impl(const void* qkv, int q_row_stride, const void* 
   if (g_decode_stream && !counters && (long long)T * Hkv * nsplit >= 1024 &&
       decode_attention_stream_fits(T, Hq, Hkv, D, page_size)) {
     rc = decode_attention_stream(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml,
-                                 T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, row_list, stream);
+                                 T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, stream);
   } else
+#define NF_DA_CALL(DD, SG) launch_split<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, sig_bias, stream)
+#define NF_DA(DD) case DD: rc = sig_bias ? NF_DA_CALL(DD, true) : NF_DA_CALL(DD, false); break;
   switch (D) {
-    case 16: rc = launch_split<16>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, stream); break;
-    case 32: rc = launch_split<32>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, stream); break;
-    case 64: rc = launch_split<64>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, stream); break;
-    case 128: rc = launch_split<128>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, stream); break;
-    case 256: rc = launch_split<256>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, stream); break;
+    NF_DA(16)
+    NF_DA(32)
+    NF_DA(64)
+    NF_DA(128)
+    NF_DA(256)
     default:
       set_error("decode attention: head_dim %d is not one of 16, 32, 64, 128, 256", D);
       return 1;
   }
+#undef NF_DA
+#undef NF_DA_CALL
   if (rc || counters) return rc;      // with counters the split kernel's last CTAs have merged
   dim3 grid(T, Hq);
   int dthreads = 32;
@@ -484,7 +521,7 @@ static int decode_attention_impl(const void* qkv, int q_row_stride, const void* 
   }
   launch_chained(decode_attention_merge_kernel<__nv_bfloat16>, grid, dim3(dthreads * groups), smem, stream,
                  (const float*)ws_acc, (const float*)ws_ml, positions, (__nv_bfloat16*)out, Hq, D, window, nsplit,
-                 dthreads, row_list);
+                 dthreads, row_list, sig_bias ? 0 : 1, turn_freq, turn_dims, interleaved);
   return check_launch("decode_attention_merge");
 }
 
@@ -511,6 +548,21 @@ extern "C" int nf_decode_attention_rows(const void* qkv, int q_row_stride, const
   return decode_attention_impl(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, out, ws_acc,
                                ws_ml, T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, nullptr, row_list,
                                stream);
+}
+
+// The further forms (see the top of this file): sig_bias float32 [Hq] or null; turn_freq float32 [turn_dims / 2] or
+// null, pairs (m, m + turn_dims / 2) or, interleaved, (2m, 2m + 1).  row_list as above, or null for all T rows.
+extern "C" int nf_decode_attention_further(const void* qkv, int q_row_stride, const void* pages,
+                                           const int* block_table, int bt_width, const int* positions,
+                                           const int* row_seg, void* out, float* ws_acc, float* ws_ml,
+                                           const int* row_list, int T, int Hq, int Hkv, int D, int page_size,
+                                           int num_pages, int window, float scale, int nsplit, const float* sig_bias,
+                                           const float* turn_freq, int turn_dims, int interleaved,
+                                           cudaStream_t stream) {
+  NF_REQUIRE(!turn_freq || (turn_dims > 0 && turn_dims % 2 == 0 && turn_dims <= D), "decode attention: %d turned numbers of %d", turn_dims, D);
+  return decode_attention_impl(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, out, ws_acc,
+                               ws_ml, T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, nullptr, row_list,
+                               stream, sig_bias, turn_freq, turn_dims, interleaved);
 }
 
 // The same in one launch: `counters` are T * Hkv ints that are zero before the call and are left

@@ -69,16 +69,16 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-// D: head size, 64 or 128.  G = Hq / Hkv <= 16 query heads share a kv head.
+// D: head size, 64 or 128.  G = Hq / Hkv <= 16 query heads share a kv head.  SIGMOID: see attention_decode.cu.
 // ws_acc [T, Hq, nsplit, D], ws_ml [T, Hq, nsplit, 2] as in attention_decode.cu.
-template <int D>
+template <int D, bool SIGMOID>
 __global__ void __launch_bounds__(kWorkers * 32, 1)
 decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride,
                                const __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table,
                                int bt_width, const int* __restrict__ positions, const int* __restrict__ row_seg,
                                float* __restrict__ ws_acc, float* __restrict__ ws_ml, int T, int Hq, int Hkv,
                                int page_size, int num_pages, int window, float scale, int nsplit,
-                               const int* __restrict__ row_list) {
+                               const int* __restrict__ row_list, const float* __restrict__ sig_bias) {
   constexpr int PIECES = D / 8;                    // 16-byte pieces of a key row
   constexpr int TILE_BYTES = kTile * D * 2;        // keys (or values) of one tile
   constexpr int STAGE_BYTES = 2 * TILE_BYTES;
@@ -236,6 +236,7 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
 #pragma unroll
       for (int i = 0; i < 4; ++i) o[db][i] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;      // rows g and g + 8; l: this lane's share
+    const float b0h = SIGMOID && g < G ? sig_bias[kvh * G + g] : 0.f, b1h = SIGMOID && g + 8 < G ? sig_bias[kvh * G + g + 8] : 0.f;
 
     for (int tile = tile0; tile < tile1; ++tile, ++used) {
       produce();                         // tile used + NS - 1 (its stage was released at the end of the last turn)
@@ -267,13 +268,22 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
           s[nb][i] = v;
           if (i < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
         }
+      float a0 = 1.f, a1 = 1.f;
+      if constexpr (SIGMOID) {
+        // exp(inf) = inf for a masked key: its weight is exactly zero
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+          for (int i = 0; i < 4; ++i) s[nb][i] = 1.f / (1.f + expf(-(s[nb][i] + (i < 2 ? b0h : b1h))));
+      } else {
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
       mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
       mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
       // every tile of a block holds at least one key of the row, so the maxima are finite
       const float n0 = fmaxf(m0, mx0), n1 = fmaxf(m1, mx1);
-      const float a0 = expf(m0 - n0), a1 = expf(m1 - n1);          // exp(-inf) = 0 on the first tile
+      a0 = expf(m0 - n0);                // exp(-inf) = 0 on the first tile
+      a1 = expf(m1 - n1);
       m0 = n0;
       m1 = n1;
       float ps0 = 0.f, ps1 = 0.f;
@@ -288,6 +298,7 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
       }
       l0 = l0 * a0 + ps0;
       l1 = l1 * a1 + ps1;
+      }  // softmax
       const unsigned pa0 = pack_bf16(s[0][0], s[0][1]), pa1 = pack_bf16(s[0][2], s[0][3]);
       const unsigned pa2 = pack_bf16(s[1][0], s[1][1]), pa3 = pack_bf16(s[1][2], s[1][3]);
       // O = O * alpha + P V: columns = head dims in blocks of 8, two blocks per ldmatrix
@@ -323,8 +334,8 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
           *reinterpret_cast<float2*>(acc + db * 8 + 2 * tq) = make_float2(o[db][2 * r], o[db][2 * r + 1]);
         if (tq == 0) {
           float* mlp = ws_ml + (((size_t)t * Hq + hq) * nsplit + split) * 2;
-          mlp[0] = r ? m1 : m0;
-          mlp[1] = r ? l1 : l0;
+          mlp[0] = SIGMOID ? 0.f : (r ? m1 : m0);
+          mlp[1] = SIGMOID ? 1.f : (r ? l1 : l0);
         }
       }
     }
@@ -332,18 +343,18 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
   cp_wait<0>();
 }
 
-template <int D>
+template <int D, bool SIGMOID>
 int launch_stream(const void* qkv, int q_row_stride, const void* pages, const int* block_table, int bt_width,
                   const int* positions, const int* row_seg, float* ws_acc, float* ws_ml, int T, int Hq, int Hkv,
                   int page_size, int num_pages, int window, float scale, int nsplit, const int* row_list,
-                  cudaStream_t stream) {
+                  const float* sig_bias, cudaStream_t stream) {
   constexpr int STAGE_BYTES = 2 * kTile * D * 2;
   constexpr int NS = kRingBytes / STAGE_BYTES < 8 ? kRingBytes / STAGE_BYTES : 8;
   const size_t smem = (size_t)kWorkers * NS * STAGE_BYTES + (size_t)(2 * T + 1) * sizeof(int);
   static bool set = false;
   if (!set) {
     const size_t most = (size_t)kWorkers * NS * STAGE_BYTES + (size_t)(2 * kMaxRows + 1) * sizeof(int);
-    cudaError_t e = cudaFuncSetAttribute(decode_attention_stream_kernel<D>,
+    cudaError_t e = cudaFuncSetAttribute(decode_attention_stream_kernel<D, SIGMOID>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most);
     NF_REQUIRE(e == cudaSuccess, "decode attention: cannot have %zu bytes of shared memory: %s", most, cudaGetErrorString(e));
     set = true;
@@ -359,9 +370,9 @@ int launch_stream(const void* qkv, int q_row_stride, const void* pages, const in
   // the longest row); workers are numbered CTA-fastest, so few blocks spread over all SMs
   const long long most_blocks = (long long)T * Hkv * nsplit;
   const int grid = (int)(most_blocks < n_sm ? most_blocks : n_sm);
-  launch_chained(decode_attention_stream_kernel<D>, dim3(grid), dim3(kWorkers * 32), smem, stream,
+  launch_chained(decode_attention_stream_kernel<D, SIGMOID>, dim3(grid), dim3(kWorkers * 32), smem, stream,
                  (const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width,
-                 positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list);
+                 positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, sig_bias);
   return check_launch("decode_attention_stream");
 }
 
@@ -384,12 +395,11 @@ int decode_attention_stream_fits(int T, int Hq, int Hkv, int D, int page_size) {
 int decode_attention_stream(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                             int bt_width, const int* positions, const int* row_seg, float* ws_acc, float* ws_ml,
                             int T, int Hq, int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                            int nsplit, const int* row_list, cudaStream_t stream) {
-  if (D == 64)
-    return launch_stream<64>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T,
-                             Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, stream);
-  return launch_stream<128>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T,
-                            Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, stream);
+                            int nsplit, const int* row_list, const float* sig_bias, cudaStream_t stream) {
+#define NF_DS(DD, SG) launch_stream<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, stream)
+  if (D == 64) return sig_bias ? NF_DS(64, true) : NF_DS(64, false);
+  return sig_bias ? NF_DS(128, true) : NF_DS(128, false);
+#undef NF_DS
 }
 
 }  // namespace nf

@@ -79,6 +79,28 @@ __global__ void rope_head_slices_kernel(T* __restrict__ q, int ldq, int heads, i
   }
 }
 
+// out[base[s] + j, :] = the cached row of segment s's position j, for every segment with base[s] >= 0 and all its
+// positions up to this step's last: a warp a row, 16-byte pieces (a row that no page holds becomes zeros).
+__global__ void __launch_bounds__(256)
+gather_cached_rows_kernel(const uint4* __restrict__ pages, const int* __restrict__ block_table, int bt_width,
+                          const int* __restrict__ seg_pos0, const int* __restrict__ seg_row0,
+                          const int* __restrict__ base, uint4* __restrict__ out, int pieces, int page_size,
+                          int num_pages, int out_rows) {
+  const int s = blockIdx.y;
+  chain_wait(pages, base);
+  const int b = base[s];
+  if (b < 0) return;
+  const int n = seg_pos0[s] + seg_row0[s + 1] - seg_row0[s];
+  const int j = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (j >= n || b + j >= out_rows) return;
+  const int lp = j / page_size;
+  const int page = lp < bt_width ? block_table[(size_t)s * bt_width + lp] : -1;
+  const bool ok = page >= 0 && page < num_pages;
+  const uint4* src = pages + ((size_t)(ok ? page : 0) * page_size + (j - lp * page_size)) * pieces;
+  uint4* dst = out + (size_t)(b + j) * pieces;
+  for (int i = lane; i < pieces; i += 32) dst[i] = ok ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
 constexpr int kLatentMaxPerLane = 16;      // R <= 512
 
 // q_abs [heads, T, R] (head-major, what the batched product leaves); q_rot read from q [T, ldq] at
@@ -192,6 +214,17 @@ extern "C" int nf_latent_append(const void* src, int lds, int col0, int R, int D
   else
     launch_chained(latent_append_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, stream, (const __nv_bfloat16*)src, lds, col0, R, Dr, w, eps, inv_freq, rot_dims, positions, row_seg, (__nv_bfloat16*)pages, block_table, bt_width, page_size, num_pages);
   return check_launch("latent_append");
+}
+
+// pages [num_pages, page_size, row_bytes], out [out_rows, row_bytes]; base int32 [S] (-1: the segment is left out).
+extern "C" int nf_gather_cached_rows(const void* pages, const int* block_table, int bt_width, const int* seg_pos0,
+                                     const int* seg_row0, const int* base, void* out, int S, int row_bytes,
+                                     int page_size, int num_pages, int max_context, int out_rows, cudaStream_t stream) {
+  if (S == 0 || out_rows == 0) return 0;
+  NF_REQUIRE(S > 0 && S <= 65535 && max_context > 0 && out_rows > 0 && row_bytes > 0 && row_bytes % 16 == 0, "gather_cached_rows: bad sizes S=%d row=%d bytes", S, row_bytes);
+  NF_REQUIRE((uintptr_t)pages % 16 == 0 && (uintptr_t)out % 16 == 0, "gather_cached_rows: rows must be 16-byte aligned");
+  launch_chained(gather_cached_rows_kernel, dim3((max_context + 7) / 8, S), dim3(256), 0, stream, (const uint4*)pages, block_table, bt_width, seg_pos0, seg_row0, base, (uint4*)out, row_bytes / 16, page_size, num_pages, out_rows);
+  return check_launch("gather_cached_rows");
 }
 
 extern "C" int nf_rope_head_slices(void* q, int ldq, int heads, int head_stride, int off, int rot_dims,

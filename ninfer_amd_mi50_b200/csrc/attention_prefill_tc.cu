@@ -30,6 +30,10 @@
 // The SIGMOID form has weights sigmoid(score + sig_bias[h]) that are not normalised over keys: no maximum, no rescaling,
 // no sum; P = 1 / (1 + 2^-(s + b)) and O is stored as it stands.
 //
+// The DENSE form reads keys and values from one row-major matrix [rows, Hkv * D keys | Hkv * D values] instead of pages
+// (what a latent cache's rows are expanded into for a prompt portion): a segment's rows lie together from kv_base[segment]
+// on, and a block is one copy an atom column.  `gate` multiplies head h's output by sigmoid(gate[row, h]).
+//
 // Everything between the roles goes through mbarriers; every wait is bounded: after a fixed
 // number of polls the kernel records a code in `g_fa_error`, tells its other warps to stop,
 // waits (bounded) for its own copies in flight, frees its tensor memory and returns.
@@ -104,13 +108,14 @@ __device__ __forceinline__ TileInfo tile_info(const int* tiles, int which, const
   return t;
 }
 
-template <int D, bool SIGMOID>
+template <int D, bool SIGMOID, bool DENSE>
 __global__ void __launch_bounds__(kFaThreads, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             const int* __restrict__ block_table, int bt_width, const int* __restrict__ positions,
                             const int* __restrict__ seg_row0, const int* __restrict__ tiles,
                             __nv_bfloat16* __restrict__ out, int Hq, int Hkv, int page_size, int num_pages,
-                            int window, float scale, const float* __restrict__ sig_bias) {
+                            int window, float scale, const float* __restrict__ sig_bias,
+                            const int* __restrict__ kv_base, const __nv_bfloat16* __restrict__ gate, int gate_ld) {
   constexpr int ATOMS = D / 64;                   // 64-column swizzle atoms across the head
   constexpr int QB = ATOMS * kAtom;               // bytes of the Q tile, of a K block, of a V block
   extern __shared__ unsigned char smem_raw[];
@@ -160,7 +165,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   // Launched chained: the zero-fill, the barriers and the tensor-memory allocation above touch
   // nothing outside the SM and ran while the kernel before this one drained; queries, keys and
   // values (and the first write of `out`) come after the wait.
-  chain_wait(block_table, positions, seg_row0, tiles);
+  chain_wait(block_table, positions, seg_row0, tiles, gate, kv_base);
 
   if (warp == 0 || warp == 10) {
     // ---- producers: warp 0 brings Q and the keys, warp 10 the values --------------------------------
@@ -172,11 +177,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       int gb = 0, issued_stage[2] = {-1, -1};
       bool ok = true, q_pending = false;
       int gq = 0;
-      const int per = kKeys / page_size;               // pages a block spans (at most 8)
+      const int per = DENSE ? 0 : kKeys / page_size;   // pages a block spans (at most 8)
       for (int which = 0; which < 2 && ok; ++which, ++gq) {
         const TileInfo t = tile_info(tiles, which, seg_row0, positions, window);
         if (t.seg < 0) break;
         const int* bt = block_table + (size_t)t.seg * bt_width;
+        const int dense_row0 = DENSE ? kv_base[t.seg] + t.kb_first : 0;
         // the pages of a block: looked up one block ahead, so that the trip to the block table
         // passes while this thread waits for a free stage
         auto lookup = [&](int blk, int* page_of) {
@@ -209,6 +215,14 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           void* full = kv ? &bars->v_full[s] : &bars->k_full[s];
           void* empty = kv ? &bars->v_empty[s] : &bars->k_empty[s];
           if (!mbar_wait(empty, ((gb >> 1) & 1) ^ 1, stop, 2, &g_fa_error)) { ok = false; break; }
+          if constexpr (DENSE) {
+            // (rows beyond the matrix read as zeros; rows of the next segment are finite and masked)
+            mbar_expect_tx(full, (unsigned)kKeys * D * 2);
+            for (int a = 0; a < ATOMS; ++a)
+              tma_load_2d(st + a * kAtom, &map_kv, (kv * Hkv + kvh) * D + 64 * a, dense_row0 + blk * kKeys, full);
+            issued_stage[s] = gb;
+            continue;
+          }
           mbar_expect_tx(full, (unsigned)n_ok * page_size * D * 2);
           for (int pi = 0; pi < per; ++pi) {
             if (page_now[pi] < 0) continue;
@@ -428,7 +442,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       }
       if (!mbar_wait(&bars->o_final, gq & 1, stop, 10, &g_fa_error)) { ok = false; break; }
       tc_fence_after();
-      const float inv = l_row > 0.f ? 1.f / l_row : 0.f;
+      float inv = l_row > 0.f ? 1.f / l_row : 0.f;
+      if (gate && row_ok) inv *= 1.f / (1.f + expf(-__bfloat162float(gate[(size_t)(t.row0 + r) * gate_ld + h])));
       __nv_bfloat16* dst = out + (size_t)(t.row0 + r) * Hq * D + (size_t)h * D + half * HD;
 #pragma unroll 1
       for (int c = 0; c < HD / 32; ++c) {
@@ -465,22 +480,23 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   }
 }
 
-template <int D, bool SIGMOID>
+template <int D, bool SIGMOID, bool DENSE>
 int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const int* block_table, int bt_width,
                       const int* positions, const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
                       int Hkv, int page_size, int num_pages, int window, float scale, const float* sig_bias,
-                      cudaStream_t stream) {
+                      const int* kv_base, const void* gate, int gate_ld, cudaStream_t stream) {
   constexpr int QB = (D / 64) * kAtom;
   const size_t smem = 1024 + (size_t)5 * QB + 2 * kAtom + sizeof(FaBarriers) + 6 * kQ * sizeof(float);
   static bool set = false;
   if (!set) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, SIGMOID, DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     NF_REQUIRE(e == cudaSuccess, "prefill attention: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     set = true;
   }
   dim3 grid(Hq, n_tiles);
-  launch_chained(prefill_attention_tc_kernel<D, SIGMOID>, grid, dim3(kFaThreads), smem, stream, mq, mkv, block_table, bt_width,
-                 positions, seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias);
+  launch_chained(prefill_attention_tc_kernel<D, SIGMOID, DENSE>, grid, dim3(kFaThreads), smem, stream, mq, mkv, block_table, bt_width,
+                 positions, seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, kv_base,
+                 (const __nv_bfloat16*)gate, gate_ld);
   return check_launch("prefill_attention_tc");
 }
 
@@ -513,7 +529,7 @@ static int attention_tc(const void* qkv, long long T, int q_row_stride, const vo
   CUtensorMap mq, mkv;
   if (int rc = make_map(&mq, qkv, T, (long long)Hq * D, kQ, q_row_stride)) return rc;
   if (int rc = make_map(&mkv, pages, (long long)num_pages * 2 * Hkv * page_size, D, page_size)) return rc;
-#define NF_TC(DD, SG) launch_prefill_tc<DD, SG>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, stream)
+#define NF_TC(DD, SG) launch_prefill_tc<DD, SG, false>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, nullptr, nullptr, 0, stream)
   if (D == 64) return sig_bias ? NF_TC(64, true) : NF_TC(64, false);
   return sig_bias ? NF_TC(128, true) : NF_TC(128, false);
 #undef NF_TC
@@ -536,6 +552,26 @@ extern "C" int nf_sigmoid_attention_tc(const void* qkv, long long T, int q_row_s
   NF_REQUIRE(sig_bias, "sigmoid attention needs its bias a head");
   return attention_tc(qkv, T, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq,
                       Hkv, D, page_size, num_pages, window, scale, sig_bias, stream);
+}
+
+// The dense form: kv [kv_rows, 2 * Hkv * D] bfloat16 row-major (keys of all heads, then values of all heads), a segment's
+// context in rows kv_base[segment] .. (int32 [segments], read only for segments that have tiles); gate bfloat16
+// [T, gate_ld] (column h: head h's gate logit) or null.
+extern "C" int nf_dense_attention_tc(const void* q, long long T, int q_row_stride, const void* kv, long long kv_rows,
+                                     const int* kv_base, const int* positions, const int* seg_row0, const int* tiles,
+                                     int n_tiles, void* out, int Hq, int Hkv, int D, float scale, const void* gate,
+                                     int gate_ld, cudaStream_t stream) {
+  if (n_tiles == 0) return 0;
+  NF_REQUIRE(n_tiles > 0 && n_tiles <= 65535 && T > 0 && kv_rows > 0 && kv_rows < (1ll << 31), "dense attention: bad sizes tiles=%d T=%lld rows=%lld", n_tiles, T, kv_rows);
+  NF_REQUIRE((D == 64 || D == 128) && Hkv > 0 && Hq % Hkv == 0, "dense attention: sizes the tensor-core kernel does not take (Hq=%d Hkv=%d D=%d)", Hq, Hkv, D);
+  NF_REQUIRE(q_row_stride % 8 == 0 && q_row_stride >= Hq * D && (uintptr_t)q % 16 == 0 && (uintptr_t)kv % 16 == 0, "dense attention: rows must be 16-byte aligned");
+  NF_REQUIRE(kv_base && (!gate || gate_ld >= Hq), "dense attention: bad arguments");
+  CUtensorMap mq, mkv;
+  if (int rc = make_map(&mq, q, T, (long long)Hq * D, kQ, q_row_stride)) return rc;
+  if (int rc = make_map(&mkv, kv, kv_rows, 2ll * Hkv * D, kKeys)) return rc;
+#define NF_TC(DD) launch_prefill_tc<DD, false, true>(mq, mkv, nullptr, 0, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, kKeys, 0, 0, scale, nullptr, kv_base, gate, gate_ld, stream)
+  return D == 64 ? NF_TC(64) : NF_TC(128);
+#undef NF_TC
 }
 
 // 0 if no tensor-core attention kernel has given up on a wait since the last call; else the code

@@ -428,13 +428,14 @@ namespace nf {
 // h[t] += table[row(t)], row(t) = (prev * mul_prev + id * mul_cur) mod buckets, or `buckets` (the
 // table's last row) for a request's first token.  The previous token of a segment's first row is
 // what the request's slot remembers (`last[slot]` = token + 1; 0: none yet); the CTA of that row
-// also leaves the segment's last token there for the next step.
-template <typename T>
+// also leaves the segment's last token there for the next step.  With `base`, the row starts as the token's
+// embedding, h[t] = base[id] * scale + table[row(t)] (h is not read).  VEC: four elements an access.
+template <typename T, bool VEC>
 __global__ void pair_hash_embed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
                                        const int* __restrict__ row_seg, const int* __restrict__ seg_row0,
                                        const int* __restrict__ seg_slot, int* __restrict__ last, long slot_stride,
                                        float* __restrict__ h, int hidden, int buckets, unsigned long long mul_prev,
-                                       unsigned long long mul_cur) {
+                                       unsigned long long mul_cur, const T* __restrict__ base, int vocab, float scale) {
   __shared__ int s_prev;
   const int t = blockIdx.x;
   chain_wait(h, last);
@@ -455,7 +456,24 @@ __global__ void pair_hash_embed_kernel(const T* __restrict__ table, const int* _
                : ((unsigned long long)prev * mul_prev + (unsigned long long)ids[t] * mul_cur) % (unsigned long long)buckets;
   const T* tr = table + (size_t)row * hidden;
   float* hr = h + (size_t)t * hidden;
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) hr[i] += to_float(tr[i]);
+  const int id = ids[t];
+  const bool known = id >= 0 && id < vocab;
+  const T* br = base ? base + (size_t)(known ? id : 0) * hidden : nullptr;
+  constexpr int W = VEC ? 4 : 1;
+  for (int i = threadIdx.x * W; i < hidden; i += blockDim.x * W) {
+    float v[W], x[W];
+    if constexpr (VEC) load4(tr + i, x); else x[0] = to_float(tr[i]);
+    if (br) {
+      if constexpr (VEC) load4(br + i, v); else v[0] = to_float(br[i]);
+#pragma unroll
+      for (int e = 0; e < W; ++e) v[e] = known ? v[e] * scale : 0.f;
+    } else {
+      if constexpr (VEC) load4(hr + i, v); else v[0] = hr[i];
+    }
+#pragma unroll
+    for (int e = 0; e < W; ++e) v[e] += x[e];
+    if constexpr (VEC) store4(hr + i, v); else hr[i] = v[0];
+  }
 }
 
 // act[m, i] = gated_act(gu[m, i] + bias[i], gu[m, inner + i] + bias[inner + i]); gu is float32 or T.
@@ -475,13 +493,18 @@ __global__ void gated_bias_act_kernel(const TI* __restrict__ gu, const float* __
 
 extern "C" int nf_pair_hash_embed(const void* table, const int* ids, const int* row_seg, const int* seg_row0,
                                   const int* seg_slot, int* last, long long slot_stride, float* h, int T, int hidden,
-                                  int buckets, long long mul_prev, long long mul_cur, int dtype, cudaStream_t stream) {
+                                  int buckets, long long mul_prev, long long mul_cur, const void* base, int vocab,
+                                  float scale, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && hidden > 0 && buckets > 0 && mul_prev >= 0 && mul_cur >= 0, "pair_hash_embed: bad arguments");
-  if (dtype == kF32)
-    launch_chained(pair_hash_embed_kernel<float>, dim3(T), dim3(row_threads(hidden)), 0, stream, (const float*)table, ids, row_seg, seg_row0, seg_slot, last, (long)slot_stride, h, hidden, buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur);
-  else
-    launch_chained(pair_hash_embed_kernel<__nv_bfloat16>, dim3(T), dim3(row_threads(hidden)), 0, stream, (const __nv_bfloat16*)table, ids, row_seg, seg_row0, seg_slot, last, (long)slot_stride, h, hidden, buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur);
+  NF_REQUIRE(!base || vocab > 0, "pair_hash_embed: an empty embedding");
+  const size_t el = dtype == kF32 ? 4 : 2;
+  const bool vec = hidden % 4 == 0 && (uintptr_t)h % 16 == 0 && (uintptr_t)table % (4 * el) == 0 && (uintptr_t)base % (4 * el) == 0;
+  const int th = row_threads(vec ? hidden / 4 : hidden);
+#define NF_PH(TT, VE) launch_chained(pair_hash_embed_kernel<TT, VE>, dim3(T), dim3(th), 0, stream, (const TT*)table, ids, row_seg, seg_row0, seg_slot, last, (long)slot_stride, h, hidden, buckets, (unsigned long long)mul_prev, (unsigned long long)mul_cur, (const TT*)base, vocab, scale)
+  if (dtype == kF32) { if (vec) NF_PH(float, true); else NF_PH(float, false); }
+  else { if (vec) NF_PH(__nv_bfloat16, true); else NF_PH(__nv_bfloat16, false); }
+#undef NF_PH
   return check_launch("pair_hash_embed");
 }
 

@@ -75,7 +75,9 @@ qk_whole_norm_append_kernel(const float* __restrict__ proj, int ld, int q_col0, 
 // Further forms: wq null - no norms; interleaved - pairs (2i, 2i + 1) instead of (i, i + rot/2); v_freq - the value is
 // turned too, over all its Dv dimensions in the same layout of pairs, pair m by pos * v_freq[m] (no magnitude).
 // The row's normed values wait in shared memory (float32) between the two passes.
-template <typename T>
+// VEC: all sizes are multiples of 4 (the turned halves too): runs of four elements an access, and the norm's
+// factors are applied where the values are read for the second time.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0, int k_col0, int v_col0,
                               const float* __restrict__ bias_q, const float* __restrict__ bias_k,
@@ -143,9 +145,12 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
       sk = fmaf(v, v, sk);
     }
   }
+  float inv_q = 1.f, inv_k = 1.f;
   if (wq) {
-    const float inv_q = 1.f / sqrtf(block_sum(sq, red) / (float)QW + eps);
-    const float inv_k = KW ? 1.f / sqrtf(block_sum(sk, red) / (float)KW + eps) : 0.f;
+    inv_q = 1.f / sqrtf(block_sum(sq, red) / (float)QW + eps);
+    inv_k = KW ? 1.f / sqrtf(block_sum(sk, red) / (float)KW + eps) : 0.f;
+  }
+  if (!VEC && wq) {
     for (int i = threadIdx.x; i < QW; i += blockDim.x) y[i] = y[i] * inv_q * wq[i];
     for (int i = threadIdx.x; i < KW; i += blockDim.x) y[QW + i] = y[QW + i] * inv_k * wk[i];
   }
@@ -178,6 +183,50 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
     T* dst = is_q ? q_out + ((size_t)t * Hq + hh) * P
                   : (krow ? krow + (size_t)(hh - Hq) * k_head_stride : nullptr);
     if (!dst) continue;
+    if constexpr (VEC) {
+      const float* w = wq ? (is_q ? wq + (size_t)hh * D : wk + (size_t)(hh - Hq) * D) : nullptr;
+      const float inv = is_q ? inv_q : inv_k;
+      auto read4 = [&](int d, float* v) {
+        load4(yy + d, v);
+        if (w) {
+          float wv[4];
+          load4(w + d, wv);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[e] = v[e] * inv * wv[e];
+        }
+      };
+      const int turned = interleaved ? half / 2 : half / 4;              // runs that hold pairs
+      for (int u = lane; u < turned + (D - rot) / 4; u += 32) {
+        float a[4], b[4], r[4], q[4];
+        if (u >= turned) {
+          const int d = rot + (u - turned) * 4;
+          read4(d, a);
+          store4(dst + d, a);
+        } else if (interleaved) {
+          const int d = u * 4;
+          read4(d, a);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float sn = sn_s[2 * u + e], cs = cs_s[2 * u + e];
+            r[2 * e] = a[2 * e] * cs - a[2 * e + 1] * sn;
+            r[2 * e + 1] = a[2 * e + 1] * cs + a[2 * e] * sn;
+          }
+          store4(dst + d, r);
+        } else {
+          const int d = u * 4;
+          read4(d, a);
+          read4(d + half, b);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float sn = sn_s[d + e], cs = cs_s[d + e];
+            r[e] = a[e] * cs - b[e] * sn;
+            q[e] = b[e] * cs + a[e] * sn;
+          }
+          store4(dst + d, r);
+          store4(dst + d + half, q);
+        }
+      }
+    } else
     for (int u = lane; u < units; u += 32) {
       if (u < half) {
         const int i0 = interleaved ? 2 * u : u, i1 = interleaved ? 2 * u + 1 : u + half;
@@ -199,6 +248,48 @@ whole_norm_rope_append_kernel(const float* __restrict__ proj, int ld, int q_col0
       T* dst = vrow + (size_t)head * v_head_stride;
       const float* src = row + v_col0 + (size_t)head * Dv;
       const float* b = bias_v ? bias_v + (size_t)head * Dv : nullptr;
+      if constexpr (VEC) {
+        auto read4 = [&](int d, float* v) {
+          load4(src + d, v);
+          if (b) {
+            float bv[4];
+            load4(b + d, bv);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] += bv[e];
+          }
+        };
+        for (int u = lane; u < Dv / 4; u += 32) {
+          float x[4], z[4], r[4], q[4];
+          const int d = u * 4;
+          if (!v_freq) {
+            read4(d, x);
+            store4(dst + d, x);
+          } else if (interleaved) {
+            read4(d, x);
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const float sn = vsn_s[2 * u + e], cs = vcs_s[2 * u + e];
+              r[2 * e] = x[2 * e] * cs - x[2 * e + 1] * sn;
+              r[2 * e + 1] = x[2 * e + 1] * cs + x[2 * e] * sn;
+            }
+            store4(dst + d, r);
+          } else if (d < vhalf) {
+            read4(d, x);
+            read4(d + vhalf, z);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float sn = vsn_s[d + e], cs = vcs_s[d + e];
+              r[e] = x[e] * cs - z[e] * sn;
+              q[e] = z[e] * cs + x[e] * sn;
+            }
+            store4(dst + d, r);
+            store4(dst + d + vhalf, q);
+          }
+        }
+        if (!rows_layout)
+          for (int d = Dv + lane; d < P; d += 32) dst[d] = from_float<T>(0.f);
+        continue;
+      }
       for (int u = lane; u < vhalf; u += 32) {
         const int i0 = interleaved ? 2 * u : u, i1 = interleaved ? 2 * u + 1 : u + vhalf;
         const float x0 = src[i0] + (b ? b[i0] : 0.f), x1 = src[i1] + (b ? b[i1] : 0.f);
@@ -334,13 +425,23 @@ extern "C" int nf_whole_norm_rope_append(const float* proj, int ld, int q_col0, 
   NF_REQUIRE(!v_freq || Dv % 2 == 0, "whole_norm_rope_append: values of %d cannot be turned in pairs", Dv);
   const size_t smem = ((size_t)(Hq + Hkv) * D + rot + (v_freq ? Dv : 0)) * sizeof(float);
   NF_REQUIRE(smem <= 200 * 1024, "whole_norm_rope_append: %d values a row do not fit shared memory", (Hq + Hkv) * D);
-  if (dtype == kF32) {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(whole_norm_rope_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_chained(whole_norm_rope_append_kernel<float>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (float*)q_out, Hq, Hkv, D, Dv, (float*)pages, block_table, bt_width, page_size, num_pages, rows_layout, P, interleaved, v_freq);
-  } else {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(whole_norm_rope_append_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch_chained(whole_norm_rope_append_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (__nv_bfloat16*)q_out, Hq, Hkv, D, Dv, (__nv_bfloat16*)pages, block_table, bt_width, page_size, num_pages, rows_layout, P, interleaved, v_freq);
-  }
+  // (which form runs depends on sizes and addresses that are the same in every step of a model)
+  const size_t el = dtype == kF32 ? 4 : 2;
+  const bool vec = ((D | Dv | P | ld | q_col0 | k_col0 | v_col0) & 3) == 0 && rot % (interleaved ? 4 : 8) == 0 &&
+                   (!v_freq || interleaved || Dv % 8 == 0) && (uintptr_t)proj % 16 == 0 && (uintptr_t)q_out % (4 * el) == 0 &&
+                   (uintptr_t)pages % (4 * el) == 0 && (uintptr_t)wq % 16 == 0 && (uintptr_t)wk % 16 == 0 &&
+                   (uintptr_t)bias_q % 16 == 0 && (uintptr_t)bias_k % 16 == 0 && (uintptr_t)bias_v % 16 == 0;
+#define NF_WN(TT, VE)                                                                                                  \
+  do {                                                                                                                \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(whole_norm_rope_append_kernel<TT, VE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    launch_chained(whole_norm_rope_append_kernel<TT, VE>, dim3(T), dim3(256), smem, stream, proj, ld, q_col0, k_col0, \
+                   v_col0, bias_q, bias_k, bias_v, wq, wk, eps, inv_freq, rot, mag, positions, row_seg, (TT*)q_out,   \
+                   Hq, Hkv, D, Dv, (TT*)pages, block_table, bt_width, page_size, num_pages, rows_layout, P,           \
+                   interleaved, v_freq);                                                                              \
+  } while (0)
+  if (dtype == kF32) { if (vec) NF_WN(float, true); else NF_WN(float, false); }
+  else { if (vec) NF_WN(__nv_bfloat16, true); else NF_WN(__nv_bfloat16, false); }
+#undef NF_WN
   return check_launch("whole_norm_rope_append");
 }
 

@@ -38,6 +38,11 @@ TUNING = {
     # prompt portions: steps with at least this many rows use the tcgen05 attention kernel (head
     # size 64 or 128), fewer the mma.sync one; a huge number turns the tensor-core kernel off
     "prefill_attention_tc_min_rows": 128,
+    # latent attention (without a rotated part) in prompt portions of at least this many rows: the cached latents are
+    # expanded into keys and values and the tcgen05 kernel runs over them, as long as those take at most
+    # `latent_expand_max_mb`; a huge number keeps every row on the latent kernel
+    "latent_expand_min_rows": 128,
+    "latent_expand_max_mb": 1024,
     "qkv_rope_fused": True,       # few bfloat16 rows: rotation and cache append in the projection's epilogue
     "router_tensor_min_rows": 128,   # router logits of more rows than this use tensor cores
     # up to this many rows, routing is a single launch (whole decode steps at 24 and 32 tokens:
@@ -513,13 +518,21 @@ def _tiles(ctx, rows_per_tile, window, keys_per_block, pair, min_rows):
 
 
 def _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out,
-                      rows: Optional[torch.Tensor], n: int) -> None:
+                      rows: Optional[torch.Tensor], n: int, sigmoid_bias: Optional[torch.Tensor] = None, turn=None) -> None:
     """The split-key decode kernels on all rows of the step (`rows` None) or on the `n` rows
-    listed in `rows` (int32 on the device); writes those rows of `out`."""
+    listed in `rows` (int32 on the device); writes those rows of `out`.  `sigmoid_bias`: sigmoid weights in the
+    softmax's place; `turn` (freq, dims, interleaved): the merge turns each head's result back."""
     nsplit = max(1, (int(ctx.max_context) + DECODE_SPLIT - 1) // DECODE_SPLIT)
     ws_acc = torch.empty((n, Hq, nsplit, D), dtype=torch.float32, device=qkv.device)
     ws_ml = torch.empty((n, Hq, nsplit, 2), dtype=torch.float32, device=qkv.device)
-    if rows is not None:
+    if sigmoid_bias is not None or turn is not None:
+        freq, dims, interleaved = turn if turn is not None else (None, 0, False)
+        _lib.call("nf_decode_attention_further", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
+                  c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg), _p(out),
+                  _p(ws_acc), _p(ws_ml), _p(rows), c_int(n), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
+                  c_int(pages.shape[0]), c_int(window), c_float(scale), c_int(nsplit), _p(sigmoid_bias), _p(freq),
+                  c_int(dims), c_int(1 if interleaved else 0), _stream())
+    elif rows is not None:
         _lib.call("nf_decode_attention_rows", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
                   c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg), _p(out),
                   _p(ws_acc), _p(ws_ml), _p(rows), c_int(n), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
@@ -539,21 +552,28 @@ def _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, windo
 
 
 def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.Tensor,
-                    block_table: torch.Tensor, page_size: int, ctx, window: int, scale: float
+                    block_table: torch.Tensor, page_size: int, ctx, window: int, scale: float, turn=None
                     ) -> torch.Tensor:
     """Causal attention of the rows' (rotated) queries in `qkv` over the cache -> [T, Hq*D].
 
     In bfloat16 a row is served according to its own segment: a segment of one row (a decoded
     token) by the split-key decode kernel, a segment of several rows (a prompt portion) by a
-    flash kernel - whatever else the step holds.  A mixed step is therefore two launches."""
+    flash kernel - whatever else the step holds.  A mixed step is therefore two launches.
+    `turn` (freq, dims, interleaved): each head's first `dims` numbers are turned by minus the row's position, in
+    the decode kernels' merge or by `turn_back`."""
     _chk(qkv, "qkv"); _chk(pages, "pages", qkv.dtype)
     T = qkv.shape[0]
+    fast = qkv.dtype == torch.bfloat16 and TUNING["bf16_attention"] != "generic"
+    if turn is not None and not (T and fast and getattr(ctx, "all_single", False) and D in DECODE_HEAD_DIMS):
+        out = paged_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale)
+        freq, dims, interleaved = turn
+        turn_back(out, ctx.positions, freq, Hq, dims, row=D, interleaved=interleaved)
+        return out
     out = torch.empty((T, Hq * D), dtype=qkv.dtype, device=qkv.device)
     if T == 0:
         return out
-    fast = qkv.dtype == torch.bfloat16 and TUNING["bf16_attention"] != "generic"
     if fast and getattr(ctx, "all_single", False) and D in DECODE_HEAD_DIMS:
-        _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out, None, T)
+        _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out, None, T, turn=turn)
         return out
     if (fast and D in PREFILL_HEAD_DIMS and getattr(ctx, "seg_len_host", None) is not None
             and getattr(ctx, "seg_pos0_host", None) is not None and qkv.shape[1] % 8 == 0):
@@ -706,8 +726,16 @@ def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: t
                           _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window),
                           c_float(scale), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), c_int(shares), _p(part_o),
                           _p(part_ml), _p(sigmoid_bias), _stream())
-            singles, n_single = ctx.one_row_tiles()
-            if n_single:
+            if sigmoid_bias is not None and gate is None and keep == 0 and D in DECODE_HEAD_DIMS:
+                # single rows: the split-key decode kernels (keys read once a key head, not once a query head)
+                rows, n_single = (None, T) if ctx.all_single else ctx.single_rows()
+                if n_single:
+                    _decode_attention(q, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out, rows, n_single,
+                                      sigmoid_bias=sigmoid_bias)
+                singles = None
+            else:
+                singles, n_single = ctx.one_row_tiles()
+            if singles is not None and n_single:
                 flash(singles, n_single, int(_lib.load().nf_prefill_attention_shares(c_int(window), c_int(int(ctx.max_context)))))
             if not ctx.all_single and (
                     sigmoid_bias is not None and gate is None and T >= TUNING["prefill_attention_tc_min_rows"]
@@ -1399,16 +1427,22 @@ def cast_rows(h: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 
 
 def pair_hash_embed(table: torch.Tensor, ctx, last: torch.Tensor, h: torch.Tensor, buckets: int, mul_prev: int,
-                    mul_cur: int) -> None:
+                    mul_cur: int, base: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """h[t] += table[(prev * mul_prev + token * mul_cur) mod buckets], or table[buckets] for a request's first
     token.  `last` int32 [slots, 1]: each request's last token + 1 (0: none), read for a segment's first row and
-    updated to the segment's last token."""
+    updated to the segment's last token.  With `base` (the token embedding, of the table's type) h[t] starts as
+    base[token] * scale instead of what it holds."""
     _chk(table, "table"); _chk(h, "h", torch.float32); _chk(last, "last", torch.int32)
+    if base is not None:
+        _chk(base, "base", table.dtype)
+        if base.shape[1] != h.shape[1]:
+            raise ValueError("pair_hash_embed: the embedding does not have the rows' width")
     if table.shape[0] != buckets + 1 or table.shape[1] != h.shape[1]:
         raise ValueError("pair_hash_embed: the table must be [buckets + 1, width]")
     _lib.call("nf_pair_hash_embed", _p(table), _p(ctx.token_ids), _p(ctx.row_seg), _p(ctx.seg_row0), _p(ctx.seg_slot),
               _p(last), c_longlong(last.stride(0)), _p(h), c_int(h.shape[0]), c_int(h.shape[1]), c_int(buckets),
-              c_longlong(mul_prev), c_longlong(mul_cur), c_int(_dt(table)), _stream())
+              c_longlong(mul_prev), c_longlong(mul_cur), _p(base), c_int(base.shape[0] if base is not None else 0),
+              c_float(scale), c_int(_dt(table)), _stream())
 
 
 LINEAR_ATTENTION_MAX_DIM = 256
@@ -1593,6 +1627,40 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, head_stride: int, rot
               _p(out), c_int(T), c_int(heads), c_int(R), c_int(Dr), c_int(page_size), c_int(pages.shape[0]),
               c_int(window), c_float(scale), c_int(_dt(q_abs)), _stream())
     return out
+
+
+def can_expand_latent(q: torch.Tensor, heads: int, D: int, Dv: int, R: int, ctx) -> bool:
+    """Whether `expanded_latent_attention` serves the step's segments of several rows."""
+    if not (q.is_cuda and q.dtype == torch.bfloat16 and TUNING["bf16_attention"] != "generic" and D == Dv and D in (64, 128)
+            and R % 8 == 0 and q.shape[1] % 8 == 0 and q.is_contiguous()
+            and ctx.seg_len_host is not None and ctx.seg_pos0_host is not None):
+        return False
+    rows = sum(n for n in ctx.seg_len_host if n > 1)
+    held = sum(p + n for p, n in zip(ctx.seg_pos0_host, ctx.seg_len_host) if n > 1)
+    return rows >= TUNING["latent_expand_min_rows"] and held * 2 * heads * D * 2 <= TUNING["latent_expand_max_mb"] << 20
+
+
+def expanded_latent_attention(q: torch.Tensor, w_kv: torch.Tensor, heads: int, D: int, pages: torch.Tensor,
+                              block_table: torch.Tensor, page_size: int, ctx, scale: float, out: torch.Tensor,
+                              gate: Optional[torch.Tensor] = None, gate_col0: int = 0) -> None:
+    """Causal softmax attention of the step's segments of several rows over a latent cache, by expanding it: the
+    segments' cached rows c (pages [n, page_size, R]) are gathered, one product with w_kv [2 * heads * D, R] (keys of
+    all heads, then values) gives every token's keys and values, and the tcgen05 kernel runs over those.  q [T, ld]
+    holds the queries in its first heads * D columns; head h's output times sigmoid(gate[t, gate_col0 + h]) (bfloat16)
+    goes to out [T, heads * D], whose rows of single-row segments are left as they are."""
+    _chk(q, "q", torch.bfloat16); _chk(w_kv, "w_kv", q.dtype); _chk(pages, "pages", q.dtype); _chk(out, "out", q.dtype)
+    R = w_kv.shape[1]
+    base, total = ctx.context_rows(2)
+    c = torch.empty((total, R), dtype=q.dtype, device=q.device)
+    _lib.call("nf_gather_cached_rows", _p(pages), _p(block_table), c_int(block_table.shape[1]), _p(ctx.seg_pos0),
+              _p(ctx.seg_row0), _p(base), _p(c), c_int(ctx.S), c_int(R * 2), c_int(page_size), c_int(pages.shape[0]),
+              c_int(int(ctx.max_context)), c_int(total), _stream())
+    kv = linear(c, w_kv)
+    tiles, n_tiles = ctx.paired_query_tiles(128, 0, 128, pair=False, min_rows=2)
+    gate_p = c_void_p(gate.data_ptr() + 2 * gate_col0) if gate is not None else None
+    _lib.call("nf_dense_attention_tc", _p(q), c_longlong(q.shape[0]), c_int(q.shape[1]), _p(kv), c_longlong(total), _p(base),
+              _p(ctx.positions), _p(ctx.seg_row0), _p(tiles), c_int(n_tiles), _p(out), c_int(heads), c_int(heads), c_int(D),
+              c_float(scale), gate_p, c_int(gate.shape[1] if gate is not None else 0), _stream())
 
 
 # ---------------------------------------------------------------------------------------

@@ -247,6 +247,40 @@ class StepContext:
         self._tiles["single"] = out
         return out
 
+    def single_rows_context(self) -> Optional["StepContext"]:
+        """The segments that bring exactly one row as a step of their own (rows in `single_rows` order), for a
+        kernel that takes whole steps; None if there are none.  Built on the host; not in graph mode."""
+        if "single_ctx" not in self._tiles:
+            rows, n = self.single_rows()
+            sub = None
+            if n:
+                segs = [s for s, m in enumerate(self.seg_len_host) if m == 1]
+                idx = self.row_seg.index_select(0, rows)
+                count = torch.arange(n + 1, dtype=torch.int32, device=self.device)
+                pos0 = [self.seg_pos0_host[s] for s in segs]
+                sub = StepContext(
+                    dtype=self.dtype, device=self.device, T=n, S=n, token_ids=self.token_ids.index_select(0, rows),
+                    positions=self.positions.index_select(0, rows), row_seg=count[:n], seg_row0=count,
+                    seg_pos0=self.seg_pos0.index_select(0, idx), seg_slot=self.seg_slot.index_select(0, idx),
+                    logit_rows=count[:0], block_tables={g: t.index_select(0, idx) for g, t in self.block_tables.items()},
+                    seg_len_host=[1] * n, seg_pos0_host=pos0, max_rows_per_seg=1, max_context=max(pos0) + 1)
+                sub.scratch["segments"] = idx
+            self._tiles["single_ctx"] = sub
+        return self._tiles["single_ctx"]
+
+    def context_rows(self, min_rows: int) -> Tuple[torch.Tensor, int]:
+        """Where each segment's whole context (what it held and what it brings) starts in a matrix that holds the
+        contexts of all segments of at least `min_rows` rows one after the other: (int32 [S], -1 for the others;
+        rows in all).  Built on the host; not in graph mode."""
+        key = ("context_rows", min_rows)
+        if key not in self._tiles:
+            base, total = [], 0
+            for n, p in zip(self.seg_len_host, self.seg_pos0_host):
+                base.append(total if n >= min_rows else -1)
+                total += p + n if n >= min_rows else 0
+            self._tiles[key] = (torch.tensor(base, dtype=torch.int32).to(self.device), total)
+        return self._tiles[key]
+
     def paired_query_tiles(self, rows_per_tile: int, window: int, keys_per_block: int,
                            pair: bool = True, min_rows: int = 1) -> Tuple[torch.Tensor, int]:
         """Query tiles two to a CTA, a heavy one with a light one.
@@ -445,6 +479,14 @@ class EmbeddingExtra(Part):
         """Add this part's rows to the float32 stream `h` [T, hidden] in place.  `state` is the
         slab [slots, *state_spec.shape] indexed by `ctx.seg_slot`, zero for a new request."""
         raise NotImplementedError
+
+    def start(self, embedding: torch.Tensor, scale: float, h: torch.Tensor, ctx: StepContext,
+              state: Optional[torch.Tensor]) -> None:
+        """h = embedding[token] * scale, and this part's rows added: what the first extra is asked for, so that
+        it may do both in one pass over the stream."""
+        from .. import kernels
+        kernels.embed_rows(embedding, ctx.token_ids, h, scale=scale)
+        self.add(h, ctx, state)
 
 
 class Mixer(Part):

@@ -47,3 +47,9 @@ class HashedPairEmbedding(EmbeddingExtra):
     def add(self, h: torch.Tensor, ctx: StepContext, state: Optional[torch.Tensor]) -> None:
         assert state is not None, "the hashed pair embedding needs a state slot"
         kernels.pair_hash_embed(self.table, ctx, state, h, self.buckets, self.mul_prev, self.mul_cur)
+
+    def start(self, embedding: torch.Tensor, scale: float, h: torch.Tensor, ctx: StepContext,
+              state: Optional[torch.Tensor]) -> None:
+        assert state is not None, "the hashed pair embedding needs a state slot"
+        kernels.pair_hash_embed(self.table, ctx, state, h, self.buckets, self.mul_prev, self.mul_cur, base=embedding,
+                                scale=scale)

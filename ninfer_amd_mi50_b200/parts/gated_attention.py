@@ -135,10 +135,7 @@ class WholeNormGatedAttention(Mixer):
 
     def check_limits(self, dtype: torch.dtype, max_context: int, page_size: int) -> None:
         if self.head_major:
-            if self.sigmoid:
-                kernels.check_head_dim(self.row)
-            else:
-                kernels.check_attention_limits(dtype, self.row, max_context, page_size)
+            kernels.check_attention_limits(dtype, self.row, max_context, page_size)
 
     # ---- forward ----------------------------------------------------------------------
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: Optional[CacheView],
@@ -169,12 +166,13 @@ class WholeNormGatedAttention(Mixer):
             o = kernels.biased_window_attention(q, H, G, P, cache.pages, cache.block_table, cache.page_size, ctx,
                                                 self.window or 0, 0, self.scale, None, sigmoid_bias=self.weight_bias)
         elif self.head_major:
+            turn = (value_freq, Dv, interleaved) if value_freq is not None else None
             o = kernels.paged_attention(q, H, G, P, cache.pages, cache.block_table, cache.page_size, ctx,
-                                        self.window or 0, self.scale)
+                                        self.window or 0, self.scale, turn=turn)
         else:
             o = kernels.talking_attention(q, H, G, D, Dv, cache.pages, cache.block_table, cache.page_size, ctx, 0,
                                           self.scale, None, None)
-        if value_freq is not None:
+        if value_freq is not None and (self.sigmoid or not self.head_major):
             kernels.turn_back(o, ctx.positions, value_freq, H, Dv, row=self.o_head, interleaved=interleaved)
         if self.has_gate:
             o = kernels.sigmoid_gate_rows(o, proj, g0)

@@ -15,7 +15,10 @@ The cache keeps one row ``[c | k_rot]`` per token (`CacheSpec` with `row_width`)
 never materialise k_h or v_h: the key projection is folded into the query
 (``q_abs_h = W_uk[h]^T q_plain_h``, so ``q_plain_h . k_h = q_abs_h . c``) and the value projection
 is applied after the weighted sum (``sum_j p_j v_h,j = W_uv[h] sum_j p_j c_j``), which is the same
-arithmetic regrouped.  Prompts, portions and decoded tokens all run this one form.
+arithmetic regrouped.  Portions of few rows and decoded tokens run this form.  For a portion of many rows it
+costs several times the arithmetic of plain attention (every score is as wide as the latent); without a rotated
+part and a sink, and with sizes the tcgen05 kernel takes, such a portion gathers its cached latents, expands
+them into keys and values by one product and runs that kernel over them.
 Norms, rotation angles, scores and softmax are 32-bit in both modes.
 
 Variants by parameter: `q_rank` None - the queries are one product of the layer's input, ``q = W_q h``, without
@@ -90,11 +93,16 @@ class LatentAttention(Mixer):
         parts = [fetch(self._n("dq" if self.q_rank else "q")), fetch(self._n("dkv"))]
         if self.has_gate:
             parts.append(fetch(self._n("gate")))
+        rows = sum(p.shape[0] for p in parts)
+        if rows % 8:                            # rows of the product stay 16-byte aligned
+            parts.append(parts[0].new_zeros((8 - rows % 8, self.hidden_size)))
         self.w_in = torch.cat(parts, dim=0).contiguous()            # rows: [c_q or q | c, k_rot | gate]
         self.w_uq = fetch(self._n("uq")) if self.q_rank else None
         self.w_o = fetch(self._n("out"))
-        self.w_uk = fetch(self._n("uk")).view(H, self.dim, self.kv_rank)                       # q_plain_h @ W_uk[h]
-        self.w_uv = fetch(self._n("uv")).view(H, self.value_dim, self.kv_rank).transpose(1, 2)  # o_h @ W_uv[h]^T
+        # one matrix, keys of all heads and then values, for expanding; its parts for the folded form
+        self.w_kv = torch.cat([fetch(self._n("uk")), fetch(self._n("uv"))], dim=0).contiguous()
+        self.w_uk = self.w_kv[:H * self.dim].view(H, self.dim, self.kv_rank)                               # q_plain_h @ W_uk[h]
+        self.w_uv = self.w_kv[H * self.dim:].view(H, self.value_dim, self.kv_rank).transpose(1, 2)          # o_h @ W_uv[h]^T
         self.q_norm = fetch(self._n("dq_norm")) if self.q_rank else None
         self.kv_norm = fetch(self._n("dkv_norm"))
         self.sink = fetch(self._n("sink")) if self.has_sink else None
@@ -129,14 +137,38 @@ class LatentAttention(Mixer):
         if cache.append:
             kernels.latent_append(proj, q_cols, R, Dr, self.kv_norm, self.eps, inv_freq, rot, ctx,
                                   cache.pages, cache.block_table, cache.page_size)
+        if (not Dr and not self.has_sink and not self.window and not (self.has_gate and not self.gate_per_head)
+                and kernels.can_expand_latent(q, H, self.dim, self.value_dim, R, ctx)):
+            return self._forward_expanded(q, proj, q_cols + R, ctx, cache)
+        o = self._folded(q, proj, q_cols + R + Dr, ctx, cache.pages, cache.block_table, cache.page_size)
+        return kernels.linear(o, self.w_o)
+
+    def _forward_expanded(self, q, proj, gate_col0: int, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+        """The segments of several rows over expanded keys and values, those of one row in the folded form."""
+        H = self.heads
+        o = torch.empty((q.shape[0], H * self.value_dim), dtype=q.dtype, device=q.device)
+        kernels.expanded_latent_attention(q, self.w_kv, H, self.dim, cache.pages, cache.block_table, cache.page_size, ctx,
+                                          self.scale, o, proj if self.has_gate else None, gate_col0)
+        sub = ctx.single_rows_context()
+        if sub is not None:
+            rows, _ = ctx.single_rows()
+            own = proj is q
+            q_s = q.index_select(0, rows)
+            proj_s = q_s if own else proj.index_select(0, rows)
+            table = cache.block_table.index_select(0, sub.scratch["segments"])
+            o.index_copy_(0, rows, self._folded(q_s, proj_s, gate_col0, sub, cache.pages, table, cache.page_size))
+        return kernels.linear(o, self.w_o)
+
+    def _folded(self, q, proj, gate_col0: int, ctx: StepContext, pages, block_table, page_size: int) -> torch.Tensor:
+        """Gated outputs [T, H * vdim] with the key projection folded into the query and the value projection
+        applied after the weighted sum."""
+        H, T = self.heads, q.shape[0]
         # the key projection folded into the query: [H, T, dim] x [H, dim, R]
         q_heads = q[:, :H * self.q_head].unflatten(1, (H, self.q_head))
         q_abs = kernels.heads_linear(q_heads[:, :, :self.dim].transpose(0, 1), self.w_uk)
-        o_lat = kernels.latent_attention(q_abs, q, self.q_head, self.dim, Dr, cache.pages, cache.block_table,
-                                         cache.page_size, ctx, self.sink, self.scale, self.window or 0)
+        o_lat = kernels.latent_attention(q_abs, q, self.q_head, self.dim, self.rot_dim, pages, block_table, page_size, ctx,
+                                         self.sink, self.scale, self.window or 0)
         v = kernels.heads_linear(o_lat, self.w_uv)                            # [H, T, vdim]
         if self.has_gate:
-            o = kernels.heads_sigmoid_gate(v, proj, q_cols + R + Dr, per_head=self.gate_per_head)
-        else:
-            o = v.transpose(0, 1).reshape(T, H * self.value_dim)
-        return kernels.linear(o, self.w_o)
+            return kernels.heads_sigmoid_gate(v, proj, gate_col0, per_head=self.gate_per_head)
+        return v.transpose(0, 1).reshape(T, H * self.value_dim)

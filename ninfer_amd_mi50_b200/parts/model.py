@@ -136,12 +136,15 @@ class DecoderModel:
                 state_of: Callable[[int], Optional[torch.Tensor]]) -> torch.Tensor:
         """Run every row of the step; return float32 logits [R, vocab] for ctx.logit_rows."""
         h = torch.empty((ctx.T, self.hidden_size * self.streams), dtype=torch.float32, device=ctx.device)
-        if self.streams == 1:
-            kernels.embed_rows(self.embedding, ctx.token_ids, h, scale=self.plan.embedding_scale)
-        else:
+        if self.streams > 1:
             kernels.embed_copies(self.embedding, ctx.token_ids, h, self.streams)
+        elif not self.embedding_extras:
+            kernels.embed_rows(self.embedding, ctx.token_ids, h, scale=self.plan.embedding_scale)
         for i, e in enumerate(self.embedding_extras):
-            e.add(h, ctx, state_of(self.extra_state_slot0 + i))
+            if i == 0:
+                e.start(self.embedding, self.plan.embedding_scale, h, ctx, state_of(self.extra_state_slot0))
+            else:
+                e.add(h, ctx, state_of(self.extra_state_slot0 + i))
         pending = None
         for run, call in enumerate(self.order):
             if call.add_vector is not None:
