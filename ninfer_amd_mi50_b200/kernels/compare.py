@@ -206,6 +206,11 @@ def work_models(s: dict, prompt: int, batch: int, context: int, design: str = ""
             own = {
                 "nf_latent_attention_mma": latent, "nf_latent_attention_generic": latent,
                 "nf_sigmoid_attention_tc": windowed,
+                "nf_dense_attention_tc": (rows_ctx * 2 * H * D * 2 + 2 * T * H * D * 2, 4.0 * H * D * pairs),
+                "nf_gather_cached_rows": (rows_ctx * R * 2 * 2, 0.0),
+                # two layers of softmax attention over everything and one of sigmoid attention in a window: their mean
+                "nf_decode_attention_further": (((2 * rows_ctx + rows_w) * 2 * H * D * 2) / 3 + 2 * T * H * D * 2,
+                                                4.0 * H * D * (2 * pairs + pairs_w) / 3),
                 # float32 sums of q, k, v in; q, key and value out
                 "nf_whole_norm_rope_append": (T * 3 * H * D * (4 + 2), 0.0),
                 "nf_turn_back": (T * H * D * (2 + 2), 0.0),
@@ -215,6 +220,7 @@ def work_models(s: dict, prompt: int, batch: int, context: int, design: str = ""
                 "nf_silu_mul": (T * (4 * W * 2 // 3) * 2 * 3, 0.0),
                 "nf_heads_sigmoid_gate": (T * H * D * 4, 0.0),
                 "nf_embed_rows": (T * W * (2 + 4), 0.0),
+                "nf_pair_hash_embed": (T * W * (2 + 2 + 4), 0.0),
             }
         table = {
             # Fetezen: keys and values of the rows' chunks once, queries in and outputs out; both products and the

@@ -156,7 +156,7 @@ class LatentAttention(Mixer):
             q_s = q.index_select(0, rows)
             proj_s = q_s if own else proj.index_select(0, rows)
             table = cache.block_table.index_select(0, sub.scratch["segments"])
-            o.index_copy_(0, rows, self._folded(q_s, proj_s, gate_col0, sub, cache.pages, table, cache.page_size))
+            o.index_copy_(0, rows.long(), self._folded(q_s, proj_s, gate_col0, sub, cache.pages, table, cache.page_size))
         return kernels.linear(o, self.w_o)
 
     def _folded(self, q, proj, gate_col0: int, ctx: StepContext, pages, block_table, page_size: int) -> torch.Tensor:

@@ -69,13 +69,16 @@ AWKWARD = model([
 ], width=100, vocab=97, eps=2e-5)
 
 # heads of 64 and 128 (the split-key decode kernel, the flash and the tcgen05 kernels), one key head for eight query
-# heads, windows around a page and two key blocks, a latent of two times 64, the whole head turned
+# heads, windows around a page and two key blocks, a latent of two times 64, latents that are expanded for prompts of
+# many rows, the whole head turned
 WIDE = model([
     layer(windowed(8, 2, 64, 64, 0.1, 65, rot=(1000.0, 64)), 64),
     layer(attention(8, 1, 128, 128, 0.05, rot=(250.0, 128), scaling=(8.0, 2.0, 16.0, 128)), 40),
     layer(latent(12, 32, 48, 128, 0.15), 64),
     layer(windowed(4, 1, 128, 128, 0.07, 130, rot=(20000.0, 32)), 48),
     layer(attention(8, 2, 64, 64, 0.06, rot=(1000.0, 32)), 64),
+    layer(latent(3, 128, 128, 64, 0.1), 40),
+    layer(latent(2, 64, 64, 96, 0.15), None),
 ], width=128, vocab=131, groups=8, scale=0.5, bigram=(1009, 3, 1))
 
 CONFIGS = {"mixed": (MIXED, 71), "awkward": (AWKWARD, 72), "wide": (WIDE, 73)}

@@ -129,11 +129,15 @@ def test_a_long_prompt_through_the_kernels_for_many_rows(folder, dtype):
     a, b = random_tokens(420, cfg["vocab"], 31), random_tokens(150, cfg["vocab"], 32)
     full = lambda i, t: {"id": i, "tokens": t, "want": list(range(len(t)))}
     steps = [{"entries": [full("a", a[:200])], "end": []},
-             {"entries": [full("a", a[200:410]), full("b", b[:140])], "end": []}]
+             {"entries": [full("b", b[:100])], "end": []},
+             # a portion of many rows beside a decoded token, then beside another portion
+             {"entries": [full("b", b[100:101]), full("a", a[200:340])], "end": []},
+             {"entries": [full("a", a[340:410]), full("b", b[101:140])], "end": []},
+             {"entries": [full("c", a[:150]), full("d", b[:1])], "end": ["c", "d"]}]
     steps += [{"entries": [full("b", b[140 + i:141 + i]), full("a", a[410 + i:411 + i])], "end": ["a", "b"] if i == 9 else []}
               for i in range(10)]
     got = run(load(d, dtype, max_context=512, page_size=64), steps)
-    for i, t in (("a", a), ("b", b)):
+    for i, t in (("a", a), ("b", b), ("c", a[:150]), ("d", b[:1])):
         ref = plain(cfg, w, t)
         compare(got[i], ref, dtype, f"{name} {i}", touchy_rows(cfg, w, t, ref))
 
@@ -271,6 +275,113 @@ def test_norm_in_groups_and_the_scaled_hashed_embedding(tmp_path, dtype, width, 
     # the first token's row is the last one of the table
     first = dict(w, bigram=torch.cat([w["bigram"][:-1], torch.zeros_like(w["bigram"][-1:])]))
     assert distance(got[:1], plain(cfg, first, toks[:1])) > 0.03
+
+
+# ---- kernels against the plain kernel -----------------------------------------------------------------
+
+def paged_case(lens, G, D, page, seed=5):
+    """Random pages for requests of `lens` tokens each, all decoding their last one."""
+    from ninfer_amd_mi50_b200.parts.base import StepContext
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    S = len(lens)
+    width = (max(lens) + page - 1) // page
+    pages = (torch.randn(S * width + 1, 2, G, page, D, device="cuda", generator=g) * 0.7).bfloat16()
+    table = torch.randperm(S * width, device="cuda", generator=g).to(torch.int32).view(S, width)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    ctx = StepContext(dtype=torch.bfloat16, device=torch.device("cuda"), T=S, S=S, token_ids=i32([0] * S),
+                      positions=i32([n - 1 for n in lens]), row_seg=i32(list(range(S))), seg_row0=i32(list(range(S + 1))),
+                      seg_pos0=i32([n - 1 for n in lens]), seg_slot=i32(list(range(S))), logit_rows=i32([0]),
+                      seg_len_host=[1] * S, seg_pos0_host=[n - 1 for n in lens], max_rows_per_seg=1, max_context=max(lens))
+    return pages, table, ctx, g
+
+
+@pytest.mark.parametrize("rows", [3, 70])
+@pytest.mark.parametrize("D", [16, 64, 128])
+@pytest.mark.parametrize("window", [0, 1, 130])
+def test_decode_kernels_with_sigmoid_weights_and_turned_values(rows, D, window):
+    """The split-key kernels - one CTA a block (few blocks), the persistent form (many) - against the plain kernel of
+    one warp a row and head on the same cache: sigmoid weights, and results turned back in the merge."""
+    from ninfer_amd_mi50_b200 import kernels
+    H, G, page = 16, 8, 16
+    lens = [1 + (37 * i) % 330 for i in range(rows)]
+    pages, table, ctx, g = paged_case(lens, G, D, page)
+    q = (torch.randn(rows, H * D, device="cuda", generator=g) * 0.7).bfloat16()
+    pb = torch.randn(H, device="cuda", generator=g)
+    freq = torch.rand(D // 2, device="cuda", generator=g)
+    sig = lambda: kernels.biased_window_attention(q, H, G, D, pages, table, page, ctx, window, 0, D ** -0.5, None, sigmoid_bias=pb)
+    soft = lambda inter: kernels.paged_attention(q, H, G, D, pages, table, page, ctx, window, D ** -0.5, turn=(freq, D, inter))
+    fast = [sig(), soft(False), soft(True)]
+    saved = kernels.TUNING["bf16_attention"]
+    try:
+        kernels.TUNING["bf16_attention"] = "generic"
+        plain_ = [sig(), soft(False), soft(True)]
+    finally:
+        kernels.TUNING["bf16_attention"] = saved
+    kernels.check_status("decode kernels")
+    for a, b in zip(fast, plain_):
+        assert (a.float() - b.float()).abs().max() <= 2e-2 * b.float().abs().max()
+
+
+@pytest.mark.parametrize("H,Dv,row,interleaved", [(3, 6, 16, False), (3, 6, 16, True), (4, 64, 64, False), (4, 64, 64, True), (5, 24, 24, True), (2, 40, 48, False)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_turning_back(H, Dv, row, interleaved, dtype):
+    from ninfer_amd_mi50_b200 import kernels
+    g = torch.Generator(device="cuda").manual_seed(1)
+    T = 9
+    o = torch.randn(T, H * row, device="cuda", generator=g).to(dtype)
+    pos = torch.randint(0, 3000, (T,), device="cuda", generator=g, dtype=torch.int32)
+    freq = torch.rand(Dv // 2, device="cuda", generator=g) * 0.1
+    x = o.double().cpu().view(T, H, row)
+    want = x.clone()
+    angles = -(pos.cpu().double()[:, None] * freq.cpu().double()[None, :])
+    want[..., :Dv] = PP.turn(x[..., :Dv], angles, Dv, interleaved)
+    kernels.turn_back(o, pos, freq, H, Dv, row=row, interleaved=interleaved)
+    tol = 2e-4 if dtype == torch.float32 else 2e-2
+    assert (o.double().cpu().view(T, H, row) - want).abs().max() <= tol
+
+
+@pytest.mark.parametrize("D,Dv,row,rot,interleaved,turned", [(16, 16, 16, 8, False, True), (16, 16, 16, 12, True, True), (24, 8, 32, 10, True, False),
+                                                             (8, 24, 32, 8, False, True), (12, 20, 32, 12, False, False), (64, 64, 64, 0, True, True)])
+@pytest.mark.parametrize("norm", [True, False])
+@pytest.mark.parametrize("layout", ["heads", "rows"])
+def test_append_in_every_form(D, Dv, row, rot, interleaved, turned, norm, layout):
+    """Norms or none, both layouts of pairs, turned values, widened heads and rows, vector and scalar accesses."""
+    from ninfer_amd_mi50_b200 import kernels
+    H, G, T, page = 4, 2, 7, 8
+    if layout == "rows":
+        row = D
+    g = torch.Generator(device="cuda").manual_seed(2)
+    pages, table, ctx, _ = paged_case([1 + 5 * i for i in range(T)], G, 16, page)
+    n = pages.shape[0]
+    pages = torch.full((n, 2, G, page, row) if layout == "heads" else (n, page, G * (D + Dv)), 9.0, device="cuda")
+    proj = torch.randn(T, H * D + G * (D + Dv), device="cuda", generator=g)
+    wq, wk = (torch.rand(H * D, device="cuda", generator=g) + 0.5, torch.rand(G * D, device="cuda", generator=g) + 0.5) if norm else (None, None)
+    freq = torch.rand(max(1, rot // 2), device="cuda", generator=g)
+    vfreq = torch.rand(Dv // 2, device="cuda", generator=g) if turned else None
+    q = kernels.whole_norm_rope_append(proj, 0, H * D, (H + G) * D, None, None, None, wq, wk, 1e-5, freq if rot else None, rot, 1.0,
+                                       H, G, D, Dv, ctx, pages, table, page, torch.float32, interleaved=interleaved,
+                                       value_freq=vfreq, row=row)
+    p = proj.double().cpu()
+    pos = ctx.positions.cpu()
+    qw, kw, v = p[:, :H * D], p[:, H * D:(H + G) * D], p[:, (H + G) * D:].reshape(T, G, Dv)
+    if norm:
+        qw, kw = PP.rms(qw, 1e-5) * wq.double().cpu(), PP.rms(kw, 1e-5) * wk.double().cpu()
+    angle = lambda f, k: pos.double()[:, None] * f.double().cpu()[None, :k]
+    spin = lambda x: PP.turn(x, angle(freq, rot // 2), rot, interleaved) if rot else x
+    qw, kw = spin(qw.reshape(T, H, D)), spin(kw.reshape(T, G, D))
+    if turned:
+        v = PP.turn(v, angle(vfreq, Dv // 2), Dv, interleaved)
+    got_q = q.double().cpu().view(T, H, row)
+    assert (got_q[..., :D] - qw).abs().max() <= 2e-4 and (got_q[..., D:] == 0).all()
+    for t in range(T):
+        pg, at = int(table[t, int(pos[t]) // page]), int(pos[t]) % page
+        if layout == "heads":
+            k_t, v_t = pages[pg, 0, :, at].double().cpu(), pages[pg, 1, :, at].double().cpu()
+            assert (k_t[:, D:] == 0).all() and (v_t[:, Dv:] == 0).all()
+        else:
+            r = pages[pg, at].double().cpu()
+            k_t, v_t = r[:G * D].view(G, D), r[G * D:].view(G, Dv)
+        assert (k_t[:, :D] - kw[t]).abs().max() <= 2e-4 and (v_t[:, :Dv] - v[t]).abs().max() <= 2e-4
 
 
 # ---- keys far away and at edges -----------------------------------------------------------------------
