@@ -229,6 +229,40 @@ def case_window_attention(tokens: int, device, single: bool = False, context: in
                                                                         D ** -0.5, slopes, gate, 0))]
 
 
+def case_sigmoid_attention(tokens: int, device, single: bool = False, context: int = 0, window: int = 1024):
+    """Sigmoid attention in a window (HQ query and key heads of 128): a prompt of `tokens` rows, or `tokens` decoded
+    rows at `context`."""
+    from . import biased_window_attention
+    D = 128
+    ctx = _one_request(tokens, device, single, context)
+    held = (context + 1) if single else tokens
+    per = (held + PAGE - 1) // PAGE
+    pages = (torch.randn(ctx.S * per + 1, 2, HQ, PAGE, D, device=device) * 0.5).bfloat16()
+    bt = torch.arange(ctx.S * per, dtype=torch.int32, device=device).view(ctx.S, per)
+    q = (torch.randn(tokens, HQ * D, device=device) * 0.5).bfloat16()
+    pb = torch.full((HQ,), -2.0, device=device)
+    return [("sigmoid_attention", lambda: biased_window_attention(q, HQ, HQ, D, pages, bt, PAGE, ctx, window, 0, D ** -0.5,
+                                                                  None, sigmoid_bias=pb))]
+
+
+def case_expanded_latent(tokens: int, device):
+    """A prompt of `tokens` rows over a latent cache (width 512, HQ heads of 128) that is expanded into keys and
+    values: gather, product, attention; and the same prompt in the folded form."""
+    from . import expanded_latent_attention, latent_attention
+    R, D = 512, 128
+    ctx = _one_request(tokens, device, False, 0)
+    ctx.seg_pos0 = torch.zeros(1, dtype=torch.int32, device=device)
+    per = (tokens + PAGE - 1) // PAGE
+    pages = (torch.randn(per + 1, PAGE, R, device=device) * 0.5).bfloat16()
+    bt = torch.arange(per, dtype=torch.int32, device=device).view(1, per)
+    q = (torch.randn(tokens, HQ * D, device=device) * 0.5).bfloat16()
+    q_abs = (torch.randn(HQ, tokens, R, device=device) * 0.2).bfloat16()
+    w_kv = (torch.randn(2 * HQ * D, R, device=device) * 0.05).bfloat16()
+    out = torch.empty(tokens, HQ * D, dtype=torch.bfloat16, device=device)
+    return [("expanded_latent_attention", lambda: expanded_latent_attention(q, w_kv, HQ, D, pages, bt, PAGE, ctx, D ** -0.5, out)),
+            ("latent_attention", lambda: latent_attention(q_abs, q, D, 0, 0, pages, bt, PAGE, ctx, None, D ** -0.5))]
+
+
 def case_talking_attention(tokens: int, device, single: bool = False, context: int = 0, chunk: int = 1536):
     """Softmax attention whose heads' scores are mixed before the softmax, over chunks of `chunk` positions and
     with a sink (HQ query and key heads of 128): a prompt of `tokens` rows, or `tokens` decoded rows at `context`."""
@@ -254,6 +288,9 @@ CASES = {
     "retention_prefill": lambda dev: case_linear_attention(2048, dev, dim=64, rotary=True),
     "window_attention_prefill": lambda dev: case_window_attention(2048, dev),
     "window_attention_decode8": lambda dev: case_window_attention(8, dev, True, 2048),
+    "sigmoid_attention_prefill": lambda dev: case_sigmoid_attention(2048, dev),
+    "sigmoid_attention_decode8": lambda dev: case_sigmoid_attention(8, dev, True, 2048),
+    "expanded_latent_prefill": lambda dev: case_expanded_latent(2048, dev),
     "latent_attention_prefill": lambda dev: case_latent_attention(2048, dev),
     "latent_attention_decode8": lambda dev: case_latent_attention(8, dev, True, 2048),
     "state_space_prefill": lambda dev: case_state_space(2048, dev),

@@ -138,6 +138,12 @@ class StepContext:
         """Every segment brings exactly one row (a decode-only step)."""
         return self.max_rows_per_seg == 1
 
+    def _ints(self, values: Sequence[int]) -> torch.Tensor:
+        """A host list as an int32 tensor on the device, without waiting for the stream (a copy from pageable
+        memory would: the launches that follow could then not run ahead of the device)."""
+        t = torch.tensor(values, dtype=torch.int32)
+        return t.pin_memory().to(self.device, non_blocking=True) if self.device.type == "cuda" else t.to(self.device)
+
     def query_tiles(self, rows_per_tile: int) -> Tuple[torch.Tensor, int]:
         """Tiles of at most `rows_per_tile` consecutive rows of one segment.
 
@@ -155,7 +161,7 @@ class StepContext:
                 flat += [s, row + r]
             row += n
         n_tiles = len(flat) // 2
-        t = torch.tensor(flat, dtype=torch.int32).reshape(n_tiles, 2).to(self.device)
+        t = self._ints(flat).view(n_tiles, 2)
         self._tiles[rows_per_tile] = (t, n_tiles)
         return t, n_tiles
 
@@ -182,7 +188,7 @@ class StepContext:
         found.sort()
         flat: List[int] = [v for _, s, r in found for v in (s, r)]
         n_tiles = len(flat) // 2
-        t = torch.tensor(flat, dtype=torch.int32).reshape(n_tiles, 2).to(self.device)
+        t = self._ints(flat).view(n_tiles, 2)
         self._tiles[key] = (t, n_tiles)
         return t, n_tiles
 
@@ -206,7 +212,7 @@ class StepContext:
         found.sort()
         flat: List[int] = [v for _, s, p in found for v in (s, p)]
         n_tiles = len(flat) // 2
-        t = torch.tensor(flat, dtype=torch.int32).reshape(n_tiles, 2).to(self.device)
+        t = self._ints(flat).view(n_tiles, 2)
         self._tiles[key] = (t, n_tiles)
         return t, n_tiles
 
@@ -225,7 +231,7 @@ class StepContext:
                     flat += [s, row, -1, -1]
                 row += n
             n_tiles = len(flat) // 4
-            self._tiles["one_row"] = ((torch.tensor(flat, dtype=torch.int32).reshape(n_tiles, 2, 2).to(self.device), n_tiles)
+            self._tiles["one_row"] = ((self._ints(flat).view(n_tiles, 2, 2), n_tiles)
                                       if n_tiles else (None, 0))
         return self._tiles["one_row"]
 
@@ -243,7 +249,7 @@ class StepContext:
             if n == 1:
                 rows.append(row)
             row += n
-        out = (torch.tensor(rows, dtype=torch.int32).to(self.device), len(rows)) if rows else (None, 0)
+        out = (self._ints(rows), len(rows)) if rows else (None, 0)
         self._tiles["single"] = out
         return out
 
@@ -278,7 +284,7 @@ class StepContext:
             for n, p in zip(self.seg_len_host, self.seg_pos0_host):
                 base.append(total if n >= min_rows else -1)
                 total += p + n if n >= min_rows else 0
-            self._tiles[key] = (torch.tensor(base, dtype=torch.int32).to(self.device), total)
+            self._tiles[key] = (self._ints(base), total)
         return self._tiles[key]
 
     def paired_query_tiles(self, rows_per_tile: int, window: int, keys_per_block: int,
@@ -290,11 +296,13 @@ class StepContext:
         (int32 [n_pairs, 2, 2] of (segment, first row), second entry (-1, -1) if there is
         none; n_pairs).  With `pair` false every CTA gets one tile, heaviest first.  Segments
         with fewer than `min_rows` rows are left out (they are served elsewhere)."""
+        if self.seg_len_host is None or self.seg_pos0_host is None:
+            raise RuntimeError("paired_query_tiles needs host segment lengths (not in graph mode)")
+        if min_rows > 1 and all(n >= min_rows for n in self.seg_len_host):
+            min_rows = 1                         # nothing is left out: one list for all who ask
         key = ("pairs", rows_per_tile, window, keys_per_block, pair, min_rows)
         if key in self._tiles:
             return self._tiles[key]
-        if self.seg_len_host is None or self.seg_pos0_host is None:
-            raise RuntimeError("paired_query_tiles needs host segment lengths (not in graph mode)")
         tiles = []
         row = 0
         for s, (n, pos0) in enumerate(zip(self.seg_len_host, self.seg_pos0_host)):
@@ -318,7 +326,7 @@ class StepContext:
             flat += [tiles[j][1], tiles[j][2]] if j > i else [-1, -1]
             i, j = i + 1, j - 1
         n_pairs = len(flat) // 4
-        t = torch.tensor(flat, dtype=torch.int32).reshape(n_pairs, 2, 2).to(self.device)
+        t = self._ints(flat).view(n_pairs, 2, 2)
         self._tiles[key] = (t, n_pairs)
         return t, n_pairs
 
