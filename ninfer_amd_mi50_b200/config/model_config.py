@@ -71,13 +71,16 @@ class LayerCall:
     `append` says whether this call writes the step's new entries into that slot;
     `state` is the index of the fixed-size state the call carries (-1: the layer's number);
     `add_vector`, if given, is (tensor name, row): that row of one of the plan's
-    `stream_vectors` is added to the residual stream right before the call.
+    `stream_vectors` is added to the residual stream right before the call;
+    `project`, if given, is the name of one of the plan's `stream_projections`: before that sum and
+    the call, the stream x becomes W [x; x0], x0 being what the stream started as (the embedding).
     """
     layer: int
     cache: int
     append: bool = True
     state: int = -1
     add_vector: Optional[Tuple[str, int]] = None
+    project: Optional[str] = None
 
     def state_slot(self) -> int:
         return self.layer if self.state < 0 else self.state
@@ -98,6 +101,8 @@ class ModelPlan:
     logit_scale: float = 1.0                                    # logits = head x * logit_scale
     # float32 tables [rows, hidden] whose rows the order may add to the stream: (name, rows)
     stream_vectors: Tuple[Tuple[str, int], ...] = ()
+    # matrices [hidden, 2 hidden] that the order may apply to the stream beside its start
+    stream_projections: Tuple[str, ...] = ()
     # parts of the "embedding" registry whose rows are added to the token embedding
     embedding_extras: Tuple[PartSpec, ...] = ()
     # residual streams a token (the blocks' arrangement reads and writes all of them; they start as

@@ -13,8 +13,8 @@
 //
 // All query heads of a group share the CTA, so keys and values are read once per kv head.
 //
-// Two further forms.  SIGMOID: a key weighs sigmoid(score + sig_bias[h]), not normalised over keys - blocks carry the
-// maximum 0 and simply add.  Turned values: the merge turns the first `turn_dims` numbers of a head's result by minus
+// Further forms.  SIGMOID: a key weighs sigmoid(score + sig_bias[h]), not normalised over keys - blocks carry the
+// maximum 0 and simply add.  CAPPED: the softmax over cap * tanh(score / cap).  Turned values: the merge turns the first `turn_dims` numbers of a head's result by minus
 // the row's position (what turn_back in qk_norm_append.cu does in a pass of its own, here on the float32 sum).
 #define NF_CHAIN_CLASS 8
 #include "common.cuh"
@@ -64,7 +64,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 // weighted sum of values are tensor-core products with the keys (values) as the 16-row
 // operand and up to 8 query heads of the group as the 8-column operand; softmax stays in
 // float32 in between.  Warp w owns keys [32 w, 32 w + 32) of the block.
-template <int D, bool SIGMOID>
+template <int D, int FORM>
 __global__ void __launch_bounds__(128)
 decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride,
                               const __nv_bfloat16* __restrict__ pages,
@@ -73,7 +73,8 @@ decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_s
                               float* __restrict__ ws_acc, float* __restrict__ ws_ml, int Hq, int Hkv,
                               int page_size, int num_pages, int window, float scale, int nsplit,
                               int* __restrict__ counters, __nv_bfloat16* __restrict__ out,
-                              const int* __restrict__ row_list, const float* __restrict__ sig_bias) {
+                              const int* __restrict__ row_list, const float* __restrict__ sig_bias, float softcap) {
+  constexpr bool SIGMOID = FORM == kFormSigmoid, CAPPED = FORM == kFormCapped;
   constexpr int LPR = D / 8;            // 16-byte pieces of one key row
   constexpr int RPL = 32 / LPR;         // key rows a warp copies at once
   constexpr int DS = D + 8;             // shared-memory row stride: 16 bytes of padding keep
@@ -198,7 +199,7 @@ decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_s
       for (int i = 0; i < 4; ++i) {
         const int r = warp * 32 + m * 16 + g + (i >> 1) * 8;
         const int h = h0 + 2 * tq + (i & 1);
-        if (h < G && r >= n0 && r < n1) sc[h * kSplit + r] = c[m][i] * scale;
+        if (h < G && r >= n0 && r < n1) sc[h * kSplit + r] = CAPPED ? cap_score(c[m][i] * scale, softcap) : c[m][i] * scale;
       }
   }
   __syncthreads();
@@ -415,26 +416,26 @@ __global__ void decode_attention_merge_kernel(const float* __restrict__ ws_acc,
   }
 }
 
-template <int D, bool SIGMOID>
+template <int D, int FORM>
 static int launch_split(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                         int bt_width, const int* positions, const int* row_seg, float* ws_acc,
                         float* ws_ml, int T, int Hq, int Hkv, int page_size, int num_pages, int window,
                         float scale, int nsplit, int* counters, void* out, const int* row_list, const float* sig_bias,
-                        cudaStream_t stream) {
+                        float softcap, cudaStream_t stream) {
   const int G = Hq / Hkv;
   const size_t smem = (size_t)2 * kSplit * (D + 8) * sizeof(__nv_bfloat16) +
                       ((size_t)G * kSplit + 4 * (G < 8 ? G : 8) * D + 2 * G) * sizeof(float);
   NF_REQUIRE(smem <= 200 * 1024, "decode attention: %d query heads per kv head need too much shared memory", G);
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
-    cudaFuncSetAttribute(decode_attention_split_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(decode_attention_split_kernel<D, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     allowed = smem;
   }
   dim3 grid(T, Hkv, nsplit);
-  launch_chained(decode_attention_split_kernel<D, SIGMOID>, grid, dim3(128), smem, stream,
+  launch_chained(decode_attention_split_kernel<D, FORM>, grid, dim3(128), smem, stream,
                  (const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width,
                  positions, row_seg, ws_acc, ws_ml, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters,
-                 (__nv_bfloat16*)out, row_list, sig_bias);
+                 (__nv_bfloat16*)out, row_list, sig_bias, softcap);
   return check_launch("decode_attention_split");
 }
 
@@ -446,7 +447,7 @@ int decode_attention_stream_fits(int T, int Hq, int Hkv, int D, int page_size);
 int decode_attention_stream(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                             int bt_width, const int* positions, const int* row_seg, float* ws_acc, float* ws_ml,
                             int T, int Hq, int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                            int nsplit, const int* row_list, const float* sig_bias, cudaStream_t stream);
+                            int nsplit, const int* row_list, const float* sig_bias, float softcap, cudaStream_t stream);
 int decode_attention_stream_status();
 int g_decode_stream = 1;
 }  // namespace nf
@@ -479,7 +480,7 @@ static int decode_attention_impl(const void* qkv, int q_row_stride, const void* 
                                  int Hq, int Hkv, int D, int page_size, int num_pages, int window,
                                  float scale, int nsplit, int* counters, const int* row_list,
                                  cudaStream_t stream, const float* sig_bias = nullptr,
-                                 const float* turn_freq = nullptr, int turn_dims = 0, int interleaved = 0) {
+                                 const float* turn_freq = nullptr, int turn_dims = 0, int interleaved = 0, float softcap = 0.f) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0 && nsplit > 0, "decode attention: bad sizes T=%d Hq=%d Hkv=%d nsplit=%d", T, Hq, Hkv, nsplit);
   NF_REQUIRE(Hkv <= 65535 && nsplit <= kMaxMergeSplits, "decode attention: too many kv heads or key blocks (context beyond %d keys)", kMaxMergeSplits * kSplit);
@@ -489,10 +490,10 @@ static int decode_attention_impl(const void* qkv, int q_row_stride, const void* 
   if (g_decode_stream && !counters && (long long)T * Hkv * nsplit >= 1024 &&
       decode_attention_stream_fits(T, Hq, Hkv, D, page_size)) {
     rc = decode_attention_stream(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml,
-                                 T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, stream);
+                                 T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, softcap, stream);
   } else
-#define NF_DA_CALL(DD, SG) launch_split<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, sig_bias, stream)
-#define NF_DA(DD) case DD: rc = sig_bias ? NF_DA_CALL(DD, true) : NF_DA_CALL(DD, false); break;
+#define NF_DA_CALL(DD, SG) launch_split<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, counters, out, row_list, sig_bias, softcap, stream)
+#define NF_DA(DD) case DD: rc = sig_bias ? NF_DA_CALL(DD, kFormSigmoid) : (softcap > 0.f ? NF_DA_CALL(DD, kFormCapped) : NF_DA_CALL(DD, kFormSoftmax)); break;
   switch (D) {
     NF_DA(16)
     NF_DA(32)
@@ -551,18 +552,19 @@ extern "C" int nf_decode_attention_rows(const void* qkv, int q_row_stride, const
 }
 
 // The further forms (see the top of this file): sig_bias float32 [Hq] or null; turn_freq float32 [turn_dims / 2] or
-// null, pairs (m, m + turn_dims / 2) or, interleaved, (2m, 2m + 1).  row_list as above, or null for all T rows.
+// null, pairs (m, m + turn_dims / 2) or, interleaved, (2m, 2m + 1); softcap > 0: scores capped.  row_list as above, or null for all T rows.
 extern "C" int nf_decode_attention_further(const void* qkv, int q_row_stride, const void* pages,
                                            const int* block_table, int bt_width, const int* positions,
                                            const int* row_seg, void* out, float* ws_acc, float* ws_ml,
                                            const int* row_list, int T, int Hq, int Hkv, int D, int page_size,
                                            int num_pages, int window, float scale, int nsplit, const float* sig_bias,
                                            const float* turn_freq, int turn_dims, int interleaved,
-                                           cudaStream_t stream) {
+                                           float softcap, cudaStream_t stream) {
+  NF_REQUIRE(!(sig_bias && softcap > 0.f), "decode attention: capped scores go with the softmax");
   NF_REQUIRE(!turn_freq || (turn_dims > 0 && turn_dims % 2 == 0 && turn_dims <= D), "decode attention: %d turned numbers of %d", turn_dims, D);
   return decode_attention_impl(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, out, ws_acc,
                                ws_ml, T, Hq, Hkv, D, page_size, num_pages, window, scale, nsplit, nullptr, row_list,
-                               stream, sig_bias, turn_freq, turn_dims, interleaved);
+                               stream, sig_bias, turn_freq, turn_dims, interleaved, softcap);
 }
 
 // The same in one launch: `counters` are T * Hkv ints that are zero before the call and are left

@@ -69,16 +69,17 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-// D: head size, 64 or 128.  G = Hq / Hkv <= 16 query heads share a kv head.  SIGMOID: see attention_decode.cu.
+// D: head size, 64 or 128.  G = Hq / Hkv <= 16 query heads share a kv head.  FORM: see attention_decode.cu.
 // ws_acc [T, Hq, nsplit, D], ws_ml [T, Hq, nsplit, 2] as in attention_decode.cu.
-template <int D, bool SIGMOID>
+template <int D, int FORM>
 __global__ void __launch_bounds__(kWorkers * 32, 1)
 decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride,
                                const __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table,
                                int bt_width, const int* __restrict__ positions, const int* __restrict__ row_seg,
                                float* __restrict__ ws_acc, float* __restrict__ ws_ml, int T, int Hq, int Hkv,
                                int page_size, int num_pages, int window, float scale, int nsplit,
-                               const int* __restrict__ row_list, const float* __restrict__ sig_bias) {
+                               const int* __restrict__ row_list, const float* __restrict__ sig_bias, float softcap) {
+  constexpr bool SIGMOID = FORM == kFormSigmoid, CAPPED = FORM == kFormCapped;
   constexpr int PIECES = D / 8;                    // 16-byte pieces of a key row
   constexpr int TILE_BYTES = kTile * D * 2;        // keys (or values) of one tile
   constexpr int STAGE_BYTES = 2 * TILE_BYTES;
@@ -264,7 +265,8 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int key = key0 + nb * 8 + 2 * tq + (i & 1);
-          const float v = (key >= k_begin && key < k_end) ? s[nb][i] * scale : -INFINITY;
+          const float sv = CAPPED ? cap_score(s[nb][i] * scale, softcap) : s[nb][i] * scale;
+          const float v = (key >= k_begin && key < k_end) ? sv : -INFINITY;
           s[nb][i] = v;
           if (i < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
         }
@@ -343,18 +345,18 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
   cp_wait<0>();
 }
 
-template <int D, bool SIGMOID>
+template <int D, int FORM>
 int launch_stream(const void* qkv, int q_row_stride, const void* pages, const int* block_table, int bt_width,
                   const int* positions, const int* row_seg, float* ws_acc, float* ws_ml, int T, int Hq, int Hkv,
                   int page_size, int num_pages, int window, float scale, int nsplit, const int* row_list,
-                  const float* sig_bias, cudaStream_t stream) {
+                  const float* sig_bias, float softcap, cudaStream_t stream) {
   constexpr int STAGE_BYTES = 2 * kTile * D * 2;
   constexpr int NS = kRingBytes / STAGE_BYTES < 8 ? kRingBytes / STAGE_BYTES : 8;
   const size_t smem = (size_t)kWorkers * NS * STAGE_BYTES + (size_t)(2 * T + 1) * sizeof(int);
   static bool set = false;
   if (!set) {
     const size_t most = (size_t)kWorkers * NS * STAGE_BYTES + (size_t)(2 * kMaxRows + 1) * sizeof(int);
-    cudaError_t e = cudaFuncSetAttribute(decode_attention_stream_kernel<D, SIGMOID>,
+    cudaError_t e = cudaFuncSetAttribute(decode_attention_stream_kernel<D, FORM>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most);
     NF_REQUIRE(e == cudaSuccess, "decode attention: cannot have %zu bytes of shared memory: %s", most, cudaGetErrorString(e));
     set = true;
@@ -370,9 +372,9 @@ int launch_stream(const void* qkv, int q_row_stride, const void* pages, const in
   // the longest row); workers are numbered CTA-fastest, so few blocks spread over all SMs
   const long long most_blocks = (long long)T * Hkv * nsplit;
   const int grid = (int)(most_blocks < n_sm ? most_blocks : n_sm);
-  launch_chained(decode_attention_stream_kernel<D, SIGMOID>, dim3(grid), dim3(kWorkers * 32), smem, stream,
+  launch_chained(decode_attention_stream_kernel<D, FORM>, dim3(grid), dim3(kWorkers * 32), smem, stream,
                  (const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width,
-                 positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, sig_bias);
+                 positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, softcap);
   return check_launch("decode_attention_stream");
 }
 
@@ -395,10 +397,11 @@ int decode_attention_stream_fits(int T, int Hq, int Hkv, int D, int page_size) {
 int decode_attention_stream(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                             int bt_width, const int* positions, const int* row_seg, float* ws_acc, float* ws_ml,
                             int T, int Hq, int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                            int nsplit, const int* row_list, const float* sig_bias, cudaStream_t stream) {
-#define NF_DS(DD, SG) launch_stream<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, stream)
-  if (D == 64) return sig_bias ? NF_DS(64, true) : NF_DS(64, false);
-  return sig_bias ? NF_DS(128, true) : NF_DS(128, false);
+                            int nsplit, const int* row_list, const float* sig_bias, float softcap, cudaStream_t stream) {
+#define NF_DS(DD, SG) launch_stream<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, row_seg, ws_acc, ws_ml, T, Hq, Hkv, page_size, num_pages, window, scale, nsplit, row_list, sig_bias, softcap, stream)
+#define NF_DS_D(DD) (sig_bias ? NF_DS(DD, kFormSigmoid) : (softcap > 0.f ? NF_DS(DD, kFormCapped) : NF_DS(DD, kFormSoftmax)))
+  return D == 64 ? NF_DS_D(64) : NF_DS_D(128);
+#undef NF_DS_D
 #undef NF_DS
 }
 

@@ -13,7 +13,8 @@
 // slope_h * (p - j) off the score of key j; `keep_first` keeps the first keys of a request
 // visible when the window has passed them (at their true positions); `gate` multiplies head h's
 // output by sigmoid(gate[t, h]); `sig_bias` (one per query head) replaces the softmax by
-// sigmoid(score + sig_bias_h), a key's own weight, not normalised over keys.
+// sigmoid(score + sig_bias_h), a key's own weight, not normalised over keys; `softcap` > 0 caps a
+// score before the mask, softcap * tanh(score / softcap).
 #include "common.cuh"
 
 namespace nf {
@@ -28,7 +29,8 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_row_stride,
                                const int* __restrict__ row_seg, T* __restrict__ out, int Hq,
                                int Hkv, int D, int page_size, int num_pages, int window,
                                float scale, const float* __restrict__ slopes, int keep_first,
-                               const float* __restrict__ gate, int gate_ld, const float* __restrict__ sig_bias) {
+                               const float* __restrict__ gate, int gate_ld, const float* __restrict__ sig_bias,
+                               float softcap) {
   extern __shared__ float q_smem[];          // [4 warps][D]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
@@ -80,7 +82,9 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int q_row_stride,
         } else {                             // a head size whose rows are not 16-byte aligned
           for (int d = 0; d < D; ++d) dot = fmaf(q[d], to_float(krow[d]), dot);
         }
-        s = dot * scale - slope * (float)(pos - j);
+        s = dot * scale;
+        if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+        s -= slope * (float)(pos - j);
       }
     }
     float p;
@@ -130,15 +134,15 @@ extern "C" int nf_paged_attention_generic(const void* qkv, int q_row_stride, con
                                           int T, int Hq, int Hkv, int D, int page_size,
                                           int num_pages, int window, float scale, int dtype,
                                           const float* slopes, int keep_first, const float* gate, int gate_ld,
-                                          const float* sig_bias, cudaStream_t stream) {
+                                          const float* sig_bias, float softcap, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attention: bad sizes T=%d Hq=%d Hkv=%d", T, Hq, Hkv);
   NF_REQUIRE(D >= 1 && D <= 256, "attention: head_dim %d must lie in [1, 256]", D);
   dim3 grid(T, (Hq + 3) / 4);
   const size_t smem = 4 * D * sizeof(float);
   if (dtype == kF32)
-    paged_attention_generic_kernel<float><<<grid, 128, smem, stream>>>((const float*)qkv, q_row_stride, (const float*)pages, block_table, bt_width, positions, row_seg, (float*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, sig_bias);
+    paged_attention_generic_kernel<float><<<grid, 128, smem, stream>>>((const float*)qkv, q_row_stride, (const float*)pages, block_table, bt_width, positions, row_seg, (float*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, sig_bias, softcap);
   else
-    paged_attention_generic_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width, positions, row_seg, (__nv_bfloat16*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, sig_bias);
+    paged_attention_generic_kernel<__nv_bfloat16><<<grid, 128, smem, stream>>>((const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width, positions, row_seg, (__nv_bfloat16*)out, Hq, Hkv, D, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, sig_bias, softcap);
   return check_launch("paged_attention_generic");
 }

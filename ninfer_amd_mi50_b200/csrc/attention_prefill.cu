@@ -17,7 +17,8 @@
 // aligned blocks that hold them are walked first, then the window's); `slopes` takes
 // slope_h * (p - j) off head h's score of key j; `gate` multiplies head h's output by
 // sigmoid(gate[row, h]).  The SIGMOID form replaces the softmax by weights sigmoid(score + sig_bias[h])
-// that are not normalised over keys: no maximum, no denominator, shares of a split row simply add.
+// that are not normalised over keys: no maximum, no denominator, shares of a split row simply add.  The CAPPED form
+// takes the softmax over cap * tanh(score / cap).
 // Steps of single rows (decode) may split a row's key blocks over several CTAs: the blocks of kept
 // first keys are one share, and every aligned group of a few window blocks (four: 256 keys, by
 // absolute position) another; each CTA leaves its unnormalised sum, maximum and denominator, and a
@@ -60,7 +61,7 @@ __device__ __forceinline__ unsigned pf_pack(float lo, float hi) {
   return *reinterpret_cast<unsigned*>(&v);
 }
 
-template <int D, bool SIGMOID>
+template <int D, int FORM>
 __global__ void __launch_bounds__(kThreads)
 prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride,
                          const __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table,
@@ -69,7 +70,8 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
                          int page_size, int num_pages, int window, float scale,
                          const float* __restrict__ slopes, int keep_first, const float* __restrict__ gate,
                          int gate_ld, int n_shares, float* __restrict__ part_o, float* __restrict__ part_ml,
-                         int kSplitBlocks, const float* __restrict__ sig_bias) {
+                         int kSplitBlocks, const float* __restrict__ sig_bias, float softcap) {
+  constexpr bool SIGMOID = FORM == kFormSigmoid, CAPPED = FORM == kFormCapped;
   constexpr int DS = D + 8;             // padded row stride in elements
   constexpr int LPR = D / 8;            // 16-byte pieces per row
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -193,7 +195,15 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_stride
     }
     // ---- scale (to base-2 exponent units), mask, online softmax ------------------------------------
     float mx[2] = {-INFINITY, -INFINITY};
-    const float sc2 = scale * kLog2e;
+    const float sc2 = CAPPED ? 1.f : scale * kLog2e;
+    if constexpr (CAPPED) {
+      // to base-2 exponent units and capped at once: c - 2 c / (1 + 2^(x * scale * 2 log2 e / cap)), c = cap log2 e
+      const float c2 = softcap * kLog2e, in2 = 2.f * scale * kLog2e / softcap;
+#pragma unroll
+      for (int n = 0; n < kBKeys / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[n][i] = c2 - __fdividef(2.f * c2, 1.f + exp2f(s[n][i] * in2));
+    }
     // every key of the block visible to every row of the warp: no mask to apply
     const bool all_visible = warp * 16 + 15 < n_rows && kb + kBKeys - 1 <= pos_first + warp * 16 &&
                              (window <= 0 || kb >= pos_first + warp * 16 + 15 - window + 1);
@@ -345,28 +355,28 @@ __global__ void split_rows_merge_kernel(const float* __restrict__ part_o, const 
   }
 }
 
-template <int D, bool SIGMOID>
+template <int D, int FORM>
 static int launch_prefill(const void* qkv, int q_row_stride, const void* pages, const int* block_table,
                           int bt_width, const int* positions, const int* seg_row0, const int* tiles,
                           int n_tiles, void* out, int Hq, int Hkv, int page_size, int num_pages, int window,
                           float scale, const float* slopes, int keep_first, const float* gate, int gate_ld,
-                          int n_shares, float* part_o, float* part_ml, const float* sig_bias, cudaStream_t stream) {
+                          int n_shares, float* part_o, float* part_ml, const float* sig_bias, float softcap, cudaStream_t stream) {
   const size_t smem = (size_t)(kBQ + 4 * kBKeys) * (D + 8) * sizeof(__nv_bfloat16);
   static bool set = false;
   if (smem > 48 * 1024 && !set) {
-    cudaFuncSetAttribute(prefill_attention_kernel<D, SIGMOID>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(prefill_attention_kernel<D, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     set = true;
   }
   dim3 grid(n_tiles, Hq, n_shares > 0 ? n_shares : 1);
-  prefill_attention_kernel<D, SIGMOID><<<grid, kThreads, smem, stream>>>(
+  prefill_attention_kernel<D, FORM><<<grid, kThreads, smem, stream>>>(
       (const __nv_bfloat16*)qkv, q_row_stride, (const __nv_bfloat16*)pages, block_table, bt_width, positions,
       seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale, slopes, keep_first, gate,
-      gate_ld, n_shares, part_o, part_ml, g_split_blocks, sig_bias);
+      gate_ld, n_shares, part_o, part_ml, g_split_blocks, sig_bias, softcap);
   if (int rc = check_launch("prefill_attention")) return rc;
   if (n_shares > 0) {
     launch_chained(split_rows_merge_kernel, dim3(n_tiles, Hq), dim3(D >= 64 ? 64 : 32), 0, stream, (const float*)part_o,
                    (const float*)part_ml, positions, tiles, (__nv_bfloat16*)out, Hq, D, window, keep_first, n_shares, gate, gate_ld,
-                   g_split_blocks, SIGMOID ? 0 : 1);
+                   g_split_blocks, FORM == kFormSigmoid ? 0 : 1);
     return check_launch("split_rows_merge");
   }
   return 0;
@@ -398,7 +408,7 @@ extern "C" int nf_set_attention_split_blocks(int n) {
 // be (-1, -1).  slopes float32 [Hq] or null; keep_first >= 0 (it counts only with a window); gate
 // float32 [T, gate_ld] (column h: head h's gate logit) or null.  n_shares > 0: every tile is one row, and a row's key blocks are split into shares (see the top of this file); n_shares must be at least
 // nf_prefill_attention_shares(window, longest context); sig_bias float32 [Hq] or null: sigmoid weights in the softmax's
-// place (then without slopes); part_o float32 [rows, Hq, n_shares, D], part_ml
+// place (then without slopes); softcap > 0: scores capped (then without slopes and sigmoid weights); part_o float32 [rows, Hq, n_shares, D], part_ml
 // [rows, Hq, n_shares, 2].
 extern "C" int nf_prefill_attention_biased(const void* qkv, int q_row_stride, const void* pages,
                                            const int* block_table, int bt_width, const int* positions,
@@ -406,7 +416,7 @@ extern "C" int nf_prefill_attention_biased(const void* qkv, int q_row_stride, co
                                            int Hkv, int D, int page_size, int num_pages, int window, float scale,
                                            const float* slopes, int keep_first, const float* gate, int gate_ld,
                                            int n_shares, float* part_o, float* part_ml, const float* sig_bias,
-                                           cudaStream_t stream) {
+                                           float softcap, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   NF_REQUIRE(n_shares >= 0 && n_shares <= 65535 && (n_shares == 0 || (part_o && part_ml)),
              "prefill attention: split rows need their workspace");
@@ -414,9 +424,10 @@ extern "C" int nf_prefill_attention_biased(const void* qkv, int q_row_stride, co
   NF_REQUIRE(q_row_stride % 8 == 0 && (uintptr_t)qkv % 16 == 0, "prefill attention: query rows must be 16-byte aligned");
   NF_REQUIRE(keep_first >= 0 && (!gate || gate_ld >= Hq), "prefill attention: bad options");
   NF_REQUIRE(!(sig_bias && slopes), "prefill attention: sigmoid weights and slopes do not go together");
+  NF_REQUIRE(!(softcap > 0.f && (sig_bias || slopes)), "prefill attention: capped scores go with the plain softmax");
   if (window <= 0) keep_first = 0;
-#define NF_PF_CALL(DD, SG) launch_prefill<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, n_shares, part_o, part_ml, sig_bias, stream)
-#define NF_PF(DD) case DD: return sig_bias ? NF_PF_CALL(DD, true) : NF_PF_CALL(DD, false);
+#define NF_PF_CALL(DD, SG) launch_prefill<DD, SG>(qkv, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, slopes, keep_first, gate, gate_ld, n_shares, part_o, part_ml, sig_bias, softcap, stream)
+#define NF_PF(DD) case DD: return sig_bias ? NF_PF_CALL(DD, kFormSigmoid) : (softcap > 0.f ? NF_PF_CALL(DD, kFormCapped) : NF_PF_CALL(DD, kFormSoftmax));
   switch (D) {
     NF_PF(16) NF_PF(32) NF_PF(48) NF_PF(64) NF_PF(80) NF_PF(96) NF_PF(112) NF_PF(128)
     default:
@@ -434,5 +445,5 @@ extern "C" int nf_prefill_attention(const void* qkv, int q_row_stride, const voi
                                     cudaStream_t stream) {
   return nf_prefill_attention_biased(qkv, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles,
                                      n_tiles, out, Hq, Hkv, D, page_size, num_pages, window, scale, nullptr, 0, nullptr,
-                                     0, 0, nullptr, nullptr, nullptr, stream);
+                                     0, 0, nullptr, nullptr, nullptr, 0.f, stream);
 }

@@ -30,6 +30,8 @@
 // The SIGMOID form has weights sigmoid(score + sig_bias[h]) that are not normalised over keys: no maximum, no rescaling,
 // no sum; P = 1 / (1 + 2^-(s + b)) and O is stored as it stands.
 //
+// The CAPPED form takes the softmax over cap * tanh(score / cap), worked out on the scores as they leave tensor memory.
+//
 // The DENSE form reads keys and values from one row-major matrix [rows, Hkv * D keys | Hkv * D values] instead of pages
 // (what a latent cache's rows are expanded into for a prompt portion): a segment's rows lie together from kv_base[segment]
 // on, and a block is one copy an atom column.  `gate` multiplies head h's output by sigmoid(gate[row, h]).
@@ -108,14 +110,16 @@ __device__ __forceinline__ TileInfo tile_info(const int* tiles, int which, const
   return t;
 }
 
-template <int D, bool SIGMOID, bool DENSE>
+template <int D, int FORM, bool DENSE>
 __global__ void __launch_bounds__(kFaThreads, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             const int* __restrict__ block_table, int bt_width, const int* __restrict__ positions,
                             const int* __restrict__ seg_row0, const int* __restrict__ tiles,
                             __nv_bfloat16* __restrict__ out, int Hq, int Hkv, int page_size, int num_pages,
                             int window, float scale, const float* __restrict__ sig_bias,
-                            const int* __restrict__ kv_base, const __nv_bfloat16* __restrict__ gate, int gate_ld) {
+                            const int* __restrict__ kv_base, const __nv_bfloat16* __restrict__ gate, int gate_ld,
+                            float softcap) {
+  constexpr bool SIGMOID = FORM == kFormSigmoid, CAPPED = FORM == kFormCapped;
   constexpr int ATOMS = D / 64;                   // 64-column swizzle atoms across the head
   constexpr int QB = ATOMS * kAtom;               // bytes of the Q tile, of a K block, of a V block
   extern __shared__ unsigned char smem_raw[];
@@ -305,7 +309,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int half = (warp - 2) >> 2;                // which half of the columns
     const int r = quad * 32 + lane;
     const unsigned lane_addr = (unsigned)(quad * 32) << 16;
-    const float sc2 = scale * kLog2e;
+    const float sc2 = CAPPED ? 1.f : scale * kLog2e;           // (capped scores are in base-2 exponent units already)
+    const float c2 = CAPPED ? softcap * kLog2e : 0.f, in2 = CAPPED ? 2.f * scale * kLog2e / softcap : 0.f;
     const float sb2 = SIGMOID ? sig_bias[h] * kLog2e : 0.f;
     constexpr int HK = kKeys / 2;                    // score columns of this thread
     constexpr int HD = D / 2;                        // output columns of this thread
@@ -341,6 +346,12 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&bars->s_empty[s]);           // the buffer may take the scores of block + 2
+        if constexpr (CAPPED) {
+          // c - 2 c / (1 + 2^(x * scale * 2 log2 e / cap)), c = cap log2 e
+#pragma unroll
+          for (int i = 0; i < HK; ++i)
+            u[i] = __float_as_uint(c2 - __fdividef(2.f * c2, 1.f + ex2(__uint_as_float(u[i]) * in2)));
+        }
         float mx = 0.f;
         if constexpr (SIGMOID) {
           if (!all_visible) {
@@ -480,23 +491,23 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   }
 }
 
-template <int D, bool SIGMOID, bool DENSE>
+template <int D, int FORM, bool DENSE>
 int launch_prefill_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const int* block_table, int bt_width,
                       const int* positions, const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq,
                       int Hkv, int page_size, int num_pages, int window, float scale, const float* sig_bias,
-                      const int* kv_base, const void* gate, int gate_ld, cudaStream_t stream) {
+                      const int* kv_base, const void* gate, int gate_ld, float softcap, cudaStream_t stream) {
   constexpr int QB = (D / 64) * kAtom;
   const size_t smem = 1024 + (size_t)5 * QB + 2 * kAtom + sizeof(FaBarriers) + 6 * kQ * sizeof(float);
   static bool set = false;
   if (!set) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, SIGMOID, DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, FORM, DENSE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     NF_REQUIRE(e == cudaSuccess, "prefill attention: cannot have %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     set = true;
   }
   dim3 grid(Hq, n_tiles);
-  launch_chained(prefill_attention_tc_kernel<D, SIGMOID, DENSE>, grid, dim3(kFaThreads), smem, stream, mq, mkv, block_table, bt_width,
+  launch_chained(prefill_attention_tc_kernel<D, FORM, DENSE>, grid, dim3(kFaThreads), smem, stream, mq, mkv, block_table, bt_width,
                  positions, seg_row0, tiles, (__nv_bfloat16*)out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, kv_base,
-                 (const __nv_bfloat16*)gate, gate_ld);
+                 (const __nv_bfloat16*)gate, gate_ld, softcap);
   return check_launch("prefill_attention_tc");
 }
 
@@ -521,7 +532,7 @@ extern "C" int nf_prefill_attention_tc_fits(int Hq, int Hkv, int D, int page_siz
 static int attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages, const int* block_table,
                         int bt_width, const int* positions, const int* seg_row0, const int* tiles, int n_tiles,
                         void* out, int Hq, int Hkv, int D, int page_size, int num_pages, int window, float scale,
-                        const float* sig_bias, cudaStream_t stream) {
+                        const float* sig_bias, float softcap, cudaStream_t stream) {
   if (n_tiles == 0) return 0;
   NF_REQUIRE(n_tiles > 0 && n_tiles <= 65535 && T > 0, "prefill attention: bad sizes tiles=%d T=%lld", n_tiles, T);
   NF_REQUIRE(nf_prefill_attention_tc_fits(Hq, Hkv, D, page_size, num_pages), "prefill attention: sizes the tensor-core kernel does not take (Hq=%d Hkv=%d D=%d page=%d)", Hq, Hkv, D, page_size);
@@ -529,9 +540,10 @@ static int attention_tc(const void* qkv, long long T, int q_row_stride, const vo
   CUtensorMap mq, mkv;
   if (int rc = make_map(&mq, qkv, T, (long long)Hq * D, kQ, q_row_stride)) return rc;
   if (int rc = make_map(&mkv, pages, (long long)num_pages * 2 * Hkv * page_size, D, page_size)) return rc;
-#define NF_TC(DD, SG) launch_prefill_tc<DD, SG, false>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, nullptr, nullptr, 0, stream)
-  if (D == 64) return sig_bias ? NF_TC(64, true) : NF_TC(64, false);
-  return sig_bias ? NF_TC(128, true) : NF_TC(128, false);
+#define NF_TC(DD, SG) launch_prefill_tc<DD, SG, false>(mq, mkv, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, page_size, num_pages, window, scale, sig_bias, nullptr, nullptr, 0, softcap, stream)
+#define NF_TC_D(DD) (sig_bias ? NF_TC(DD, kFormSigmoid) : (softcap > 0.f ? NF_TC(DD, kFormCapped) : NF_TC(DD, kFormSoftmax)))
+  return D == 64 ? NF_TC_D(64) : NF_TC_D(128);
+#undef NF_TC_D
 #undef NF_TC
 }
 
@@ -541,7 +553,7 @@ extern "C" int nf_prefill_attention_tc(const void* qkv, long long T, int q_row_s
                                        int Hkv, int D, int page_size, int num_pages, int window, float scale,
                                        cudaStream_t stream) {
   return attention_tc(qkv, T, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq,
-                      Hkv, D, page_size, num_pages, window, scale, nullptr, stream);
+                      Hkv, D, page_size, num_pages, window, scale, nullptr, 0.f, stream);
 }
 
 extern "C" int nf_sigmoid_attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages,
@@ -551,7 +563,18 @@ extern "C" int nf_sigmoid_attention_tc(const void* qkv, long long T, int q_row_s
                                        const float* sig_bias, cudaStream_t stream) {
   NF_REQUIRE(sig_bias, "sigmoid attention needs its bias a head");
   return attention_tc(qkv, T, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq,
-                      Hkv, D, page_size, num_pages, window, scale, sig_bias, stream);
+                      Hkv, D, page_size, num_pages, window, scale, sig_bias, 0.f, stream);
+}
+
+// Softmax over softcap * tanh(score / softcap).
+extern "C" int nf_capped_attention_tc(const void* qkv, long long T, int q_row_stride, const void* pages,
+                                      const int* block_table, int bt_width, const int* positions,
+                                      const int* seg_row0, const int* tiles, int n_tiles, void* out, int Hq, int Hkv,
+                                      int D, int page_size, int num_pages, int window, float scale, float softcap,
+                                      cudaStream_t stream) {
+  NF_REQUIRE(softcap > 0.f, "capped attention needs a positive cap");
+  return attention_tc(qkv, T, q_row_stride, pages, block_table, bt_width, positions, seg_row0, tiles, n_tiles, out, Hq,
+                      Hkv, D, page_size, num_pages, window, scale, nullptr, softcap, stream);
 }
 
 // The dense form: kv [kv_rows, 2 * Hkv * D] bfloat16 row-major (keys of all heads, then values of all heads), a segment's
@@ -569,7 +592,7 @@ extern "C" int nf_dense_attention_tc(const void* q, long long T, int q_row_strid
   CUtensorMap mq, mkv;
   if (int rc = make_map(&mq, q, T, (long long)Hq * D, kQ, q_row_stride)) return rc;
   if (int rc = make_map(&mkv, kv, kv_rows, 2ll * Hkv * D, kKeys)) return rc;
-#define NF_TC(DD) launch_prefill_tc<DD, false, true>(mq, mkv, nullptr, 0, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, kKeys, 0, 0, scale, nullptr, kv_base, gate, gate_ld, stream)
+#define NF_TC(DD) launch_prefill_tc<DD, kFormSoftmax, true>(mq, mkv, nullptr, 0, positions, seg_row0, tiles, n_tiles, out, Hq, Hkv, kKeys, 0, 0, scale, nullptr, kv_base, gate, gate_ld, 0.f, stream)
   return D == 64 ? NF_TC(64) : NF_TC(128);
 #undef NF_TC
 }

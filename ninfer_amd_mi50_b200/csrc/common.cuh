@@ -233,6 +233,12 @@ __device__ __forceinline__ float gated_act(float g, float u, int kind, float lim
     return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
   return g / (1.f + expf(-g)) * u;
 }
+// Forms of the attention kernels: the softmax, weights sigmoid(score + bias) that are not normalised over keys, and
+// the softmax over scores that were capped, score <- cap * tanh(score / cap).
+enum AttentionForm : int { kFormSoftmax = 0, kFormSigmoid = 1, kFormCapped = 2 };
+// cap * tanh(x / cap) as cap - 2 cap / (1 + exp(2 x / cap)): the error is a few float32 roundings of cap itself.
+__device__ __forceinline__ float cap_score(float x, float cap) { return cap - __fdividef(2.f * cap, 1.f + expf(2.f * x / cap)); }
+
 __device__ __forceinline__ float relu_square(float v) { const float r = fmaxf(v, 0.f); return r * r; }
 __device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }
 __device__ __forceinline__ float gated_act(float g, float u, const GatedActParams& a) {

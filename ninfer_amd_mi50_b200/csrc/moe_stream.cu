@@ -96,6 +96,7 @@ struct MsArgs {
   float* topk_w;               // [T, k]
   float* extra_out;            // [T, extra] or null
   int* inv;                    // [M] pair -> sorted position
+  const float* rbias;          // [E] added to the experts' logits, or null
   int extra, norm_topk;
   // a shared expert inside the launch (n_shared > 0, with routing only): its intermediate features in
   // n_shared chunks of I, packed like n_shared further experts; chunk c takes rows M + c T .. of act and Y
@@ -275,7 +276,7 @@ __device__ __forceinline__ void ms_route(const MsArgs& p, float* scratch, int* s
       int* table = p.work + kMsTable;
       for (int tt = warp; tt < p.T; tt += kMsConsumers)
         select_token(p.logits + (size_t)tt * rows, 1, lg + warp * p.E, tt, p.E, p.extra, p.k, p.norm_topk, nullptr,
-                     sw, p.extra > 0 ? sext : nullptr, lane, chosen);
+                     sw, p.extra > 0 ? sext : nullptr, lane, chosen, p.rbias);
       consumers_sync();
       // stable counting sort of the pairs by expert
       for (int e2 = warp; e2 < p.E; e2 += kMsConsumers) {
@@ -853,7 +854,7 @@ extern "C" int nf_moe_stream(const void* X, int ldx, const void* W13, long long 
                              void* act, void* Y, int M, int T, int H, int I, int E, int k, const int* offsets,
                              const int* order, const int* active, int n_mapped, int* work, int q,
                              int smem_bytes, const float* Wr, int extra, int norm_topk, float* logits, int* topk_idx,
-                             float* topk_w, float* extra_out, int* inv, const void* Ws13, long long gss13,
+                             float* topk_w, float* extra_out, int* inv, const float* rbias, const void* Ws13, long long gss13,
                              const void* Ws2, long long gss2, int n_shared, float* cw, int* cinv,
                              int act_kind, float act_limit, float act_alpha, cudaStream_t stream) {
   if (M == 0) return 0;
@@ -876,7 +877,7 @@ extern "C" int nf_moe_stream(const void* X, int ldx, const void* W13, long long 
   a.offsets = offsets; a.order = order; a.active = active; a.work = work;
   a.gs13 = gs13; a.gs2 = gs2;
   a.Wr = Wr; a.logits = logits; a.topk_idx = topk_idx; a.topk_w = topk_w; a.extra_out = extra_out; a.inv = inv;
-  a.extra = Wr ? extra : 0; a.norm_topk = norm_topk;
+  a.extra = Wr ? extra : 0; a.norm_topk = norm_topk; a.rbias = Wr ? rbias : nullptr;
   a.Ws13 = (const __nv_bfloat16*)Ws13; a.Ws2 = (const __nv_bfloat16*)Ws2; a.gss13 = gss13; a.gss2 = gss2;
   a.n_shared = n_shared; a.cw = n_shared ? cw : nullptr; a.cinv = n_shared ? cinv : nullptr;
   a.ldx = ldx; a.M = M; a.T = T; a.H = H; a.I = I; a.E = E; a.k = k; a.n_mapped = n_mapped;

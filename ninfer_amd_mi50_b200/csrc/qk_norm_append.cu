@@ -360,27 +360,29 @@ turn_back_kernel(T* __restrict__ o, const int* __restrict__ positions, const flo
   }
 }
 
-// out[t, c] = o[t, c] * sigmoid(g[t, g_col0 + c]): an output gate element by element; the gate's
-// logits are float32 sums or of the rows' type.
+// out[t, h * Dv + d] = o[t, h * P + d] * sigmoid(g[t, g_col0 + h * Dv + d]), d < Dv: an output gate element by element;
+// the gate's logits are float32 sums or of the rows' type.  P > Dv: the heads of o are wider than the values (widened
+// with zeros), out has the values side by side.
 // VEC: four consecutive elements a thread, each operand's run in one access.
 template <typename T, typename TG, bool VEC>
 __global__ void sigmoid_gate_rows_kernel(const T* __restrict__ o, const TG* __restrict__ g, int ldg, int g_col0,
-                                         T* __restrict__ out, int width) {
+                                         T* __restrict__ out, int width, int Dv, int P) {
   const int t = blockIdx.y;
   chain_wait(o, g);
   constexpr int W = VEC ? 4 : 1;
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * W;
   if (c >= width) return;
+  const size_t oc = P == Dv ? (size_t)t * width + c : (size_t)t * (width / Dv) * P + (size_t)(c / Dv) * P + c % Dv;
   if constexpr (VEC) {
     float ov[4], gv[4];
-    load4(o + (size_t)t * width + c, ov);
+    load4(o + oc, ov);
     load4(g + (size_t)t * ldg + g_col0 + c, gv);
 #pragma unroll
     for (int e = 0; e < 4; ++e) ov[e] = ov[e] * (1.f / (1.f + expf(-gv[e])));
     store4(out + (size_t)t * width + c, ov);
   } else {
     const float gv = to_float(g[(size_t)t * ldg + g_col0 + c]);
-    out[(size_t)t * width + c] = from_float<T>(to_float(o[(size_t)t * width + c]) * (1.f / (1.f + expf(-gv))));
+    out[(size_t)t * width + c] = from_float<T>(to_float(o[oc]) * (1.f / (1.f + expf(-gv))));
   }
 }
 
@@ -466,21 +468,22 @@ extern "C" int nf_turn_back(void* o, const int* positions, const float* freq, in
   return check_launch("turn_back");
 }
 
-// o, out [T, width] of `dtype`; g [T, ldg] float32 (g_dtype 0) or of `dtype`.
+// out [T, width] of `dtype`, width = heads * Dv; o [T, heads * P]; g [T, ldg] float32 (g_dtype 0) or of `dtype`.
 extern "C" int nf_sigmoid_gate_rows(const void* o, const void* g, int g_dtype, int ldg, int g_col0, void* out, int T,
-                                    int width, int dtype, cudaStream_t stream) {
+                                    int width, int Dv, int P, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && T <= 65535 * 1024 && width > 0 && g_col0 >= 0 && g_col0 + width <= ldg, "sigmoid_gate_rows: bad sizes");
+  NF_REQUIRE(Dv > 0 && width % Dv == 0 && P >= Dv, "sigmoid_gate_rows: heads of %d in rows of %d, %d in all", Dv, P, width);
   NF_REQUIRE(g_dtype == kF32 || g_dtype == dtype, "sigmoid_gate_rows: the gate is float32 or of the rows' type");
   const size_t tsize = dtype == kF32 ? 4 : 2, gsize = g_dtype == kF32 ? 4 : 2;
-  const bool vec = width % 4 == 0 && ldg % 4 == 0 && g_col0 % 4 == 0 && (uintptr_t)o % (4 * tsize) == 0 &&
+  const bool vec = width % 4 == 0 && (P == Dv || (P % 4 == 0 && Dv % 4 == 0)) && ldg % 4 == 0 && g_col0 % 4 == 0 && (uintptr_t)o % (4 * tsize) == 0 &&
                    (uintptr_t)out % (4 * tsize) == 0 && (uintptr_t)g % (4 * gsize) == 0;
   for (int t0 = 0; t0 < T; t0 += 65535) {
     const int rows = T - t0 < 65535 ? T - t0 : 65535;
     const dim3 grid(((vec ? width / 4 : width) + 255) / 256, rows);
-    const size_t off = (size_t)t0 * width, goff = (size_t)t0 * ldg;
+    const size_t off = (size_t)t0 * width, ooff = (size_t)t0 * (width / Dv) * P, goff = (size_t)t0 * ldg;
 #define NF_SG(TT, TG_, V) \
-  launch_chained(sigmoid_gate_rows_kernel<TT, TG_, V>, grid, dim3(256), 0, stream, (const TT*)o + off, (const TG_*)g + goff, ldg, g_col0, (TT*)out + off, width)
+  launch_chained(sigmoid_gate_rows_kernel<TT, TG_, V>, grid, dim3(256), 0, stream, (const TT*)o + ooff, (const TG_*)g + goff, ldg, g_col0, (TT*)out + off, width, Dv, P)
     if (dtype == kF32) { if (vec) NF_SG(float, float, true); else NF_SG(float, float, false); }
     else if (g_dtype == kF32) { if (vec) NF_SG(__nv_bfloat16, float, true); else NF_SG(__nv_bfloat16, float, false); }
     else { if (vec) NF_SG(__nv_bfloat16, __nv_bfloat16, true); else NF_SG(__nv_bfloat16, __nv_bfloat16, false); }

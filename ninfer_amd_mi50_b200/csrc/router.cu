@@ -47,7 +47,7 @@ router_logits_kernel(const T* __restrict__ x, const float* __restrict__ wr, int 
 __global__ void __launch_bounds__(128)
 router_select_kernel(const float* __restrict__ logits, long tok_stride, long exp_stride, int n_tokens,
                      int E, int extra, int k, int norm_topk, int* __restrict__ topk_idx,
-                     float* __restrict__ topk_w, float* __restrict__ extra_out) {
+                     float* __restrict__ topk_w, float* __restrict__ extra_out, const float* __restrict__ bias) {
   extern __shared__ float smem[];      // [4 warps][E]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
@@ -55,7 +55,7 @@ router_select_kernel(const float* __restrict__ logits, long tok_stride, long exp
   if (t >= n_tokens) return;
   // logits[t, e] sits at t * tok_stride + e * exp_stride (either may be the unit stride)
   select_token(logits + (size_t)t * tok_stride, exp_stride, smem + warp * E, t, E, extra, k, norm_topk,
-               topk_idx, topk_w, extra_out, lane);
+               topk_idx, topk_w, extra_out, lane, nullptr, bias);
 }
 
 __global__ void __launch_bounds__(128)
@@ -107,7 +107,8 @@ router_fused_kernel(const T* __restrict__ x, const float* __restrict__ wr, int n
                     int E, int extra, int k, int norm_topk, float* __restrict__ logits,
                     int* __restrict__ topk_idx, float* __restrict__ topk_w, float* __restrict__ extra_out,
                     int* __restrict__ offsets, int* __restrict__ order, int* __restrict__ inv,
-                    int* __restrict__ active, int n_active_max, int* __restrict__ ticket) {
+                    int* __restrict__ active, int n_active_max, int* __restrict__ ticket,
+                    const float* __restrict__ bias) {
   extern __shared__ float xs[];        // [hidden]; the last block reuses it
   __shared__ int s_last;
   const int rows = E + extra;
@@ -162,7 +163,7 @@ router_fused_kernel(const T* __restrict__ x, const float* __restrict__ wr, int n
   float* lg = xs;                                   // [8 warps][E]
   for (int tt = warp; tt < n_tokens; tt += 8)
     select_token(logits + (size_t)tt * rows, 1, lg + warp * E, tt, E, extra, k, norm_topk, topk_idx, topk_w,
-                 extra_out, lane);
+                 extra_out, lane, nullptr, bias);
   __threadfence_block();
   __syncthreads();
   int* counts = reinterpret_cast<int*>(xs);         // [E + 1], then the pairs' experts
@@ -203,7 +204,7 @@ router_cluster_kernel(const T* __restrict__ x, const float* __restrict__ wr, int
                       int E, int extra, int k, int norm_topk, float* __restrict__ logits_out,
                       int* __restrict__ topk_idx, float* __restrict__ topk_w, float* __restrict__ extra_out,
                       int* __restrict__ offsets, int* __restrict__ order, int* __restrict__ inv,
-                      int* __restrict__ active, int n_active_max) {
+                      int* __restrict__ active, int n_active_max, const float* __restrict__ bias) {
   extern __shared__ __align__(16) float rs[];
   const int rows = E + extra;
   const int n = n_tokens * k;
@@ -306,7 +307,7 @@ router_cluster_kernel(const T* __restrict__ x, const float* __restrict__ wr, int
   // ---- CTA 0: selection for every token, then the plan, all in shared memory --------------------
   for (int tt = warp; tt < n_tokens; tt += 8)
     select_token<false>(lg_all + (size_t)tt * rows, 1, sel + warp * E, tt, E, extra, k, norm_topk, topk_idx, topk_w,
-                        extra_out, lane, chosen);
+                        extra_out, lane, chosen, bias);
   __syncthreads();
   for (int e = warp; e < E; e += 8) {
     int running = 0;
@@ -447,10 +448,11 @@ static int launch_logits_t(const void* x, const float* wr, int T_, int hidden, i
   return launch_logits<T, 1>(x, wr, T_, hidden, rows, logits, stream);
 }
 
-// logits: float32 scratch [T, E + extra], also an output (the raw router logits).
+// logits: float32 scratch [T, E + extra], also an output (the raw router logits).  Here and below: bias float32 [E] or
+// null is added to the experts' logits where they are chosen among.
 extern "C" int nf_router_topk(const void* x, const float* wr, int T, int hidden, int E, int extra,
                               int k, int norm_topk, float* logits, int* topk_idx, float* topk_w,
-                              float* extra_out, int dtype, cudaStream_t stream) {
+                              float* extra_out, const float* bias, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && hidden > 0 && E > 0 && k > 0 && k <= E && extra >= 0, "router: bad sizes T=%d hidden=%d E=%d k=%d", T, hidden, E, k);
   NF_REQUIRE((size_t)hidden * 4 <= 200 * 1024, "router: hidden=%d needs more shared memory than a block has", hidden);
@@ -458,7 +460,7 @@ extern "C" int nf_router_topk(const void* x, const float* wr, int T, int hidden,
   int rc = dtype == kF32 ? launch_logits_t<float>(x, wr, T, hidden, E + extra, logits, stream)
                          : launch_logits_t<__nv_bfloat16>(x, wr, T, hidden, E + extra, logits, stream);
   if (rc) return rc;
-  router_select_kernel<<<(T + 3) / 4, 128, (size_t)4 * E * sizeof(float), stream>>>(logits, E + extra, 1, T, E, extra, k, norm_topk, topk_idx, topk_w, extra_out);
+  router_select_kernel<<<(T + 3) / 4, 128, (size_t)4 * E * sizeof(float), stream>>>(logits, E + extra, 1, T, E, extra, k, norm_topk, topk_idx, topk_w, extra_out, bias);
   return check_launch("router_select");
 }
 
@@ -467,7 +469,7 @@ extern "C" int nf_router_topk(const void* x, const float* wr, int T, int hidden,
 extern "C" int nf_router_fused(const void* x, const float* wr, int T, int hidden, int E, int extra, int k,
                                int norm_topk, float* logits, int* topk_idx, float* topk_w,
                                float* extra_out, int* offsets, int* order, int* inv, int* active,
-                               int n_active_max, int* ticket, int dtype, cudaStream_t stream) {
+                               int n_active_max, int* ticket, const float* bias, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && T <= 65535 && hidden > 0 && E > 0 && k > 0 && k <= E && extra >= 0, "router: bad sizes T=%d hidden=%d E=%d k=%d", T, hidden, E, k);
   size_t words = (size_t)hidden;
@@ -479,10 +481,10 @@ extern "C" int nf_router_fused(const void* x, const float* wr, int T, int hidden
   dim3 grid((E + extra + 7) / 8, T);
   if (dtype == kF32) {
     if (smem > allowed_f) { cudaFuncSetAttribute(router_fused_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); allowed_f = smem; }
-    launch_chained(router_fused_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, wr, T, hidden, E, extra, k, norm_topk, logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max, ticket);
+    launch_chained(router_fused_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, wr, T, hidden, E, extra, k, norm_topk, logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max, ticket, bias);
   } else {
     if (smem > allowed_b) { cudaFuncSetAttribute(router_fused_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); allowed_b = smem; }
-    launch_chained(router_fused_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, wr, T, hidden, E, extra, k, norm_topk, logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max, ticket);
+    launch_chained(router_fused_kernel<__nv_bfloat16>, grid, dim3(256), smem, stream, (const __nv_bfloat16*)x, wr, T, hidden, E, extra, k, norm_topk, logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max, ticket, bias);
   }
   return check_launch("router_fused");
 }
@@ -498,7 +500,7 @@ extern "C" int nf_router_cluster_fits(int T, int hidden, int E, int extra, int k
 extern "C" int nf_router_cluster(const void* x, const float* wr, int T, int hidden, int E, int extra, int k,
                                  int norm_topk, float* logits, int* topk_idx, float* topk_w,
                                  float* extra_out, int* offsets, int* order, int* inv, int* active,
-                                 int n_active_max, int dtype, cudaStream_t stream) {
+                                 int n_active_max, const float* bias, int dtype, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && hidden > 0 && E > 0 && k > 0 && k <= E && extra >= 0, "router: bad sizes T=%d hidden=%d E=%d k=%d", T, hidden, E, k);
   NF_REQUIRE(nf_router_cluster_fits(T, hidden, E, extra, k), "router: sizes too large for the cluster kernel");
@@ -535,11 +537,11 @@ extern "C" int nf_router_cluster(const void* x, const float* wr, int T, int hidd
   if (dtype == kF32) {
     if (smem > allowed_f) { cudaFuncSetAttribute(router_cluster_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); allowed_f = smem; }
     e = cudaLaunchKernelEx(&cfg, router_cluster_kernel<float>, (const float*)x, wr, T, hidden, E, extra, k, norm_topk,
-                           logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max);
+                           logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max, bias);
   } else {
     if (smem > allowed_b) { cudaFuncSetAttribute(router_cluster_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); allowed_b = smem; }
     e = cudaLaunchKernelEx(&cfg, router_cluster_kernel<__nv_bfloat16>, (const __nv_bfloat16*)x, wr, T, hidden, E, extra, k,
-                           norm_topk, logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max);
+                           norm_topk, logits, topk_idx, topk_w, extra_out, offsets, order, inv, active, n_active_max, bias);
   }
   if (e != cudaSuccess) note_launch_error(e);
   return check_launch("router_cluster");
@@ -550,11 +552,11 @@ extern "C" int nf_router_cluster(const void* x, const float* wr, int T, int hidd
 // (1, T)).
 extern "C" int nf_router_select(const float* logits, long long tok_stride, long long exp_stride, int T,
                                 int E, int extra, int k, int norm_topk, int* topk_idx, float* topk_w,
-                                float* extra_out, cudaStream_t stream) {
+                                float* extra_out, const float* bias, cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(T > 0 && E > 0 && k > 0 && k <= E && extra >= 0, "router: bad sizes T=%d E=%d k=%d", T, E, k);
   NF_REQUIRE((size_t)4 * E * 4 <= 48 * 1024, "router: %d experts are more than the selection kernel holds (3072)", E);
-  launch_chained(router_select_kernel, dim3((T + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), stream, logits, (long)tok_stride, (long)exp_stride, T, E, extra, k, norm_topk, topk_idx, topk_w, extra_out);
+  launch_chained(router_select_kernel, dim3((T + 3) / 4), dim3(128), (size_t)4 * E * sizeof(float), stream, logits, (long)tok_stride, (long)exp_stride, T, E, extra, k, norm_topk, topk_idx, topk_w, extra_out, bias);
   return check_launch("router_select");
 }
 

@@ -50,12 +50,14 @@ __device__ __forceinline__ float lane_dot(const float* __restrict__ xs, const fl
 // GLOBAL: the logits are in global memory, written by other blocks of this launch (read past
 // L1); otherwise they are in this block's shared memory.  `chosen`, if given, also receives the
 // k selected experts of the token as 16-bit ids (shared memory, for a plan in the same block).
+// `bias` (float32 [E] or null) is added to the experts' logits.
 // topk_idx / topk_w / extra_out may be null: a block that only needs `chosen`.
 template <bool GLOBAL = true>
 __device__ __forceinline__ void select_token(const float* row, long exp_stride, float* lg, int t, int E,
                                              int extra, int k, int norm_topk, int* __restrict__ topk_idx,
                                              float* __restrict__ topk_w, float* __restrict__ extra_out,
-                                             int lane, unsigned short* chosen = nullptr) {
+                                             int lane, unsigned short* chosen = nullptr,
+                                             const float* __restrict__ bias = nullptr) {
   const bool sigmoid_scores = (norm_topk & 2) != 0;
   norm_topk &= 1;
   // (the further rows' logits are asked for together with the experts', and stored once those are in)
@@ -68,7 +70,7 @@ __device__ __forceinline__ void select_token(const float* row, long exp_stride, 
   float mx = -INFINITY;
   for (int e = lane; e < E; e += 32) {
     const float* p = row + (size_t)e * exp_stride;
-    const float v = GLOBAL ? __ldcg(p) : *p;
+    const float v = (GLOBAL ? __ldcg(p) : *p) + (bias ? bias[e] : 0.f);
     lg[e] = v;
     mx = fmaxf(mx, v);
   }

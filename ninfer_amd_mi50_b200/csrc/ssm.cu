@@ -4,7 +4,8 @@
 //    its slot, so a portion of a prompt (or one decoded token) starts from what the portion
 //    before it left; before a sequence's start the inputs are zeros (the slot is zeroed when a
 //    request is admitted).  Every output is independent of the others, so all rows of a step
-//    run in parallel; a second, small kernel then shifts the step's last inputs into the slot.
+//    run in parallel; a second, small kernel then shifts the step's last inputs into the slot (in a
+//    step of single rows a thread shifts its own channels itself).
 //
 //  * the selective scan  S_t = exp(-exp(A_log) dt_t) S_{t-1} + dt_t B_t x_t^T,
 //    y_t = S_t^T C_t + D x_t  with dt_t = softplus(raw_t + dt_bias), per head; S is [N, P]
@@ -27,19 +28,19 @@ constexpr int kMaxTaps = 8;
 // neighbouring threads read neighbouring numbers)   u from this step's rows
 // of `src` (column col0 + c), from the slot for positions before the step, zero before the start.
 // A thread owns VE consecutive channels (VE > 1: 16 bytes a load and a store, columns 16-byte aligned).
-template <typename T, int VE>
+template <typename T, int VE, bool SINGLE>
 __global__ void causal_conv_silu_kernel(const T* __restrict__ src, int lds, int col0, int C,
                                         const float* __restrict__ taps, const float* __restrict__ bias, int K,
-                                        const float* __restrict__ state, long slot_stride,
+                                        float* __restrict__ state, long slot_stride,
                                         const int* __restrict__ row_seg, const int* __restrict__ seg_row0,
                                         const int* __restrict__ seg_slot, T* __restrict__ out, int T_rows) {
   const int t = blockIdx.x;
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VE;
-  chain_wait(src);
+  chain_wait(src, state);
   if (c >= C) return;
   const int seg = row_seg[t];
   const int r0 = seg_row0[seg];
-  const float* st = state + (size_t)seg_slot[seg] * slot_stride;      // [K - 1][C]
+  float* st = state + (size_t)seg_slot[seg] * slot_stride;            // [K - 1][C]
   float acc[VE];
 #pragma unroll
   for (int e = 0; e < VE; ++e) acc[e] = bias ? bias[c + e] : 0.f;
@@ -55,6 +56,10 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ src, int lds, int 
       const int i = (K - 1) - (r0 - r);  // slot row: K - 2 is the token just before the step
 #pragma unroll
       for (int e = 0; e < VE; ++e) u[e] = i >= 0 ? st[(size_t)i * C + c + e] : 0.f;
+    }
+    if (SINGLE && j > 0) {               // the slot's row j - 1 becomes what its row j (or this row) held
+#pragma unroll
+      for (int e = 0; e < VE; ++e) st[(size_t)(j - 1) * C + c + e] = u[e];
     }
 #pragma unroll
     for (int e = 0; e < VE; ++e) acc[e] = fmaf(taps[(size_t)j * C + c + e], u[e], acc[e]);     // taps are [K][C] here
@@ -331,27 +336,32 @@ using namespace nf;
 
 extern "C" void nf_set_scan_columns(int columns) { g_scan_columns = columns; }
 
+// single != 0: every segment brings one row.
 extern "C" int nf_causal_conv_silu(const void* src, int lds, int col0, int C, const float* taps, const float* bias,
                                    int K, float* state, long long slot_stride, const int* row_seg,
-                                   const int* seg_row0, const int* seg_slot, void* out, int T, int S, int dtype,
+                                   const int* seg_row0, const int* seg_slot, void* out, int T, int S, int single, int dtype,
                                    cudaStream_t stream) {
   if (T == 0) return 0;
   NF_REQUIRE(K >= 1 && K <= kMaxTaps, "causal_conv: %d taps (1..%d)", K, kMaxTaps);
   NF_REQUIRE(C > 0 && col0 >= 0 && col0 + C <= lds, "causal_conv: bad columns");
   const dim3 sgrid(S, (C + 255) / 256);
-  if (dtype == kF32) {
-    if (C % 4 == 0 && lds % 4 == 0 && col0 % 4 == 0)
-      launch_chained(causal_conv_silu_kernel<float, 4>, dim3(T, (C / 4 + 127) / 128), dim3(128), 0, stream, (const float*)src, lds, col0, C, taps, bias, K, (const float*)state, (long)slot_stride, row_seg, seg_row0, seg_slot, (float*)out, T);
-    else
-      launch_chained(causal_conv_silu_kernel<float, 1>, dim3(T, (C + 255) / 256), dim3(256), 0, stream, (const float*)src, lds, col0, C, taps, bias, K, (const float*)state, (long)slot_stride, row_seg, seg_row0, seg_slot, (float*)out, T);
-    if (K > 1) launch_chained(conv_state_shift_kernel<float>, sgrid, dim3(256), 0, stream, (const float*)src, lds, col0, C, K, state, (long)slot_stride, seg_row0, seg_slot);
-  } else {
-    if (C % 8 == 0 && lds % 8 == 0 && col0 % 8 == 0)
-      launch_chained(causal_conv_silu_kernel<__nv_bfloat16, 8>, dim3(T, (C / 8 + 127) / 128), dim3(128), 0, stream, (const __nv_bfloat16*)src, lds, col0, C, taps, bias, K, (const float*)state, (long)slot_stride, row_seg, seg_row0, seg_slot, (__nv_bfloat16*)out, T);
-    else
-      launch_chained(causal_conv_silu_kernel<__nv_bfloat16, 1>, dim3(T, (C + 255) / 256), dim3(256), 0, stream, (const __nv_bfloat16*)src, lds, col0, C, taps, bias, K, (const float*)state, (long)slot_stride, row_seg, seg_row0, seg_slot, (__nv_bfloat16*)out, T);
-    if (K > 1) launch_chained(conv_state_shift_kernel<__nv_bfloat16>, sgrid, dim3(256), 0, stream, (const __nv_bfloat16*)src, lds, col0, C, K, state, (long)slot_stride, seg_row0, seg_slot);
-  }
+  const int ve = dtype == kF32 ? 4 : 8;
+  const bool vec = C % ve == 0 && lds % ve == 0 && col0 % ve == 0;
+#define NF_CONV(TT, VE, SI)                                                                                              \
+  launch_chained(causal_conv_silu_kernel<TT, VE, SI>, dim3(T, (C / (VE) + (VE > 1 ? 127 : 255)) / (VE > 1 ? 128 : 256)),  \
+                 dim3(VE > 1 ? 128 : 256), 0, stream, (const TT*)src, lds, col0, C, taps, bias, K, state, (long)slot_stride, \
+                 row_seg, seg_row0, seg_slot, (TT*)out, T)
+#define NF_CONV_T(TT, VE)                                                                                                \
+  do {                                                                                                                  \
+    if (vec) { if (single) NF_CONV(TT, VE, true); else NF_CONV(TT, VE, false); }                                        \
+    else { if (single) NF_CONV(TT, 1, true); else NF_CONV(TT, 1, false); }                                              \
+    if (K > 1 && !single)                                                                                               \
+      launch_chained(conv_state_shift_kernel<TT>, sgrid, dim3(256), 0, stream, (const TT*)src, lds, col0, C, K, state,   \
+                     (long)slot_stride, seg_row0, seg_slot);                                                            \
+  } while (0)
+  if (dtype == kF32) NF_CONV_T(float, 4); else NF_CONV_T(__nv_bfloat16, 8);
+#undef NF_CONV_T
+#undef NF_CONV
   return check_launch("causal_conv_silu");
 }
 

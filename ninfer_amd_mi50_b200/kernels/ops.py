@@ -519,20 +519,22 @@ def _tiles(ctx, rows_per_tile, window, keys_per_block, pair, min_rows):
 
 
 def _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out,
-                      rows: Optional[torch.Tensor], n: int, sigmoid_bias: Optional[torch.Tensor] = None, turn=None) -> None:
+                      rows: Optional[torch.Tensor], n: int, sigmoid_bias: Optional[torch.Tensor] = None, turn=None,
+                      softcap: float = 0.0) -> None:
     """The split-key decode kernels on all rows of the step (`rows` None) or on the `n` rows
     listed in `rows` (int32 on the device); writes those rows of `out`.  `sigmoid_bias`: sigmoid weights in the
-    softmax's place; `turn` (freq, dims, interleaved): the merge turns each head's result back."""
+    softmax's place; `turn` (freq, dims, interleaved): the merge turns each head's result back; `softcap` > 0: the
+    softmax is over softcap * tanh(score / softcap)."""
     nsplit = max(1, (int(ctx.max_context) + DECODE_SPLIT - 1) // DECODE_SPLIT)
     ws_acc = torch.empty((n, Hq, nsplit, D), dtype=torch.float32, device=qkv.device)
     ws_ml = torch.empty((n, Hq, nsplit, 2), dtype=torch.float32, device=qkv.device)
-    if sigmoid_bias is not None or turn is not None:
+    if sigmoid_bias is not None or turn is not None or softcap > 0.0:
         freq, dims, interleaved = turn if turn is not None else (None, 0, False)
         _lib.call("nf_decode_attention_further", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
                   c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg), _p(out),
                   _p(ws_acc), _p(ws_ml), _p(rows), c_int(n), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
                   c_int(pages.shape[0]), c_int(window), c_float(scale), c_int(nsplit), _p(sigmoid_bias), _p(freq),
-                  c_int(dims), c_int(1 if interleaved else 0), _stream())
+                  c_int(dims), c_int(1 if interleaved else 0), c_float(softcap), _stream())
     elif rows is not None:
         _lib.call("nf_decode_attention_rows", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
                   c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg), _p(out),
@@ -553,20 +555,20 @@ def _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, windo
 
 
 def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.Tensor,
-                    block_table: torch.Tensor, page_size: int, ctx, window: int, scale: float, turn=None
-                    ) -> torch.Tensor:
+                    block_table: torch.Tensor, page_size: int, ctx, window: int, scale: float, turn=None,
+                    softcap: float = 0.0) -> torch.Tensor:
     """Causal attention of the rows' (rotated) queries in `qkv` over the cache -> [T, Hq*D].
 
     In bfloat16 a row is served according to its own segment: a segment of one row (a decoded
     token) by the split-key decode kernel, a segment of several rows (a prompt portion) by a
     flash kernel - whatever else the step holds.  A mixed step is therefore two launches.
     `turn` (freq, dims, interleaved): each head's first `dims` numbers are turned by minus the row's position, in
-    the decode kernels' merge or by `turn_back`."""
+    the decode kernels' merge or by `turn_back`.  `softcap` > 0: the softmax is over softcap * tanh(score / softcap)."""
     _chk(qkv, "qkv"); _chk(pages, "pages", qkv.dtype)
     T = qkv.shape[0]
     fast = qkv.dtype == torch.bfloat16 and TUNING["bf16_attention"] != "generic"
     if turn is not None and not (T and fast and getattr(ctx, "all_single", False) and D in DECODE_HEAD_DIMS):
-        out = paged_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale)
+        out = paged_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, softcap=softcap)
         freq, dims, interleaved = turn
         turn_back(out, ctx.positions, freq, Hq, dims, row=D, interleaved=interleaved)
         return out
@@ -574,7 +576,8 @@ def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.T
     if T == 0:
         return out
     if fast and getattr(ctx, "all_single", False) and D in DECODE_HEAD_DIMS:
-        _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out, None, T, turn=turn)
+        _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out, None, T, turn=turn,
+                          softcap=softcap)
         return out
     if (fast and D in PREFILL_HEAD_DIMS and getattr(ctx, "seg_len_host", None) is not None
             and getattr(ctx, "seg_pos0_host", None) is not None and qkv.shape[1] % 8 == 0):
@@ -583,19 +586,26 @@ def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.T
             rows, n_single = ctx.single_rows()
             if n_single:
                 _decode_attention(qkv, Hq, Hkv, D, pages, block_table, page_size, ctx, window, scale, out,
-                                  rows, n_single)
+                                  rows, n_single, softcap=softcap)
                 min_rows = 2
         if (T >= TUNING["prefill_attention_tc_min_rows"] and qkv.is_contiguous() and pages.is_contiguous()
                 and _lib.load().nf_prefill_attention_tc_fits(c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
                                                             c_longlong(pages.shape[0]))):
             # tcgen05 / TMEM / TMA: tiles of 128 rows, blocks of 128 keys
             tiles, n_tiles = _tiles(ctx, 128, window, 128, False, min_rows)
-            _lib.call("nf_prefill_attention_tc", _p(qkv), c_longlong(T), c_int(qkv.shape[1]), _p(pages),
+            name, more = ("nf_capped_attention_tc", (c_float(softcap),)) if softcap > 0.0 else ("nf_prefill_attention_tc", ())
+            _lib.call(name, _p(qkv), c_longlong(T), c_int(qkv.shape[1]), _p(pages),
                       _p(block_table), c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0),
                       _p(tiles), c_int(n_tiles), _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
-                      c_int(pages.shape[0]), c_int(window), c_float(scale), _stream())
+                      c_int(pages.shape[0]), c_int(window), c_float(scale), *more, _stream())
             return out
         tiles, n_tiles = _tiles(ctx, PREFILL_TILE_ROWS, window, PREFILL_KEY_BLOCK, True, min_rows)
+        if softcap > 0.0:
+            _lib.call("nf_prefill_attention_biased", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
+                      c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0), _p(tiles), c_int(n_tiles), _p(out),
+                      c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window), c_float(scale),
+                      None, c_int(0), None, c_int(0), c_int(0), None, None, None, c_float(softcap), _stream())
+            return out
         _lib.call("nf_prefill_attention", _p(qkv), c_int(qkv.shape[1]), _p(pages), _p(block_table),
                   c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0), _p(tiles),
                   c_int(n_tiles), _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
@@ -605,7 +615,7 @@ def paged_attention(qkv: torch.Tensor, Hq: int, Hkv: int, D: int, pages: torch.T
               _p(block_table), c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg),
               _p(out), c_int(T), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size),
               c_int(pages.shape[0]), c_int(window), c_float(scale), c_int(_dt(qkv)), None, c_int(0), None,
-              c_int(0), None, _stream())
+              c_int(0), None, c_float(softcap), _stream())
     return out
 
 
@@ -678,14 +688,17 @@ def turn_back(o: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, H: i
               c_int(1 if interleaved else 0), c_int(_dt(o)), _stream())
 
 
-def sigmoid_gate_rows(o: torch.Tensor, g_src: torch.Tensor, g_col0: int) -> torch.Tensor:
+def sigmoid_gate_rows(o: torch.Tensor, g_src: torch.Tensor, g_col0: int, heads: int = 1, Dv: int = 0) -> torch.Tensor:
     """o [T, n] times sigmoid(g_src[:, g_col0 : g_col0 + n]) element by element; the gate's logits are float32
-    or of o's type."""
+    or of o's type.  With `heads` and `Dv`, o is [T, heads * P] with heads wider than their Dv values (P >= Dv): the
+    values alone are taken, the result is [T, heads * Dv]."""
     _chk(o, "o"); _chk(g_src, "g_src")
-    T, n = o.shape
-    out = torch.empty_like(o)
+    T, P = o.shape[0], o.shape[1] // heads
+    Dv = Dv or P
+    n = heads * Dv
+    out = torch.empty((T, n), dtype=o.dtype, device=o.device)
     _lib.call("nf_sigmoid_gate_rows", _p(o), _p(g_src), c_int(_dt(g_src)), c_int(g_src.shape[1]), c_int(g_col0), _p(out),
-              c_int(T), c_int(n), c_int(_dt(o)), _stream())
+              c_int(T), c_int(n), c_int(Dv), c_int(P), c_int(_dt(o)), _stream())
     return out
 
 
@@ -726,7 +739,7 @@ def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: t
                           c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.seg_row0), _p(tiles), c_int(n_tiles),
                           _p(out), c_int(Hq), c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window),
                           c_float(scale), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), c_int(shares), _p(part_o),
-                          _p(part_ml), _p(sigmoid_bias), _stream())
+                          _p(part_ml), _p(sigmoid_bias), c_float(0.0), _stream())
             if sigmoid_bias is not None and gate is None and keep == 0 and D in DECODE_HEAD_DIMS:
                 # single rows: the split-key decode kernels (keys read once a key head, not once a query head)
                 rows, n_single = (None, T) if ctx.all_single else ctx.single_rows()
@@ -757,7 +770,7 @@ def biased_window_attention(q: torch.Tensor, Hq: int, Hkv: int, D: int, pages: t
     _lib.call("nf_paged_attention_generic", _p(q), c_int(q.shape[1]), _p(pages), _p(block_table),
               c_int(block_table.shape[1]), _p(ctx.positions), _p(ctx.row_seg), _p(out), c_int(T), c_int(Hq),
               c_int(Hkv), c_int(D), c_int(page_size), c_int(pages.shape[0]), c_int(window), c_float(scale),
-              c_int(_dt(q)), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), _p(sigmoid_bias), _stream())
+              c_int(_dt(q)), _p(slopes), c_int(keep), gate_p, c_int(gate_ld), _p(sigmoid_bias), c_float(0.0), _stream())
     return out
 
 
@@ -796,14 +809,16 @@ def _route_flags(norm_topk: bool, scoring: str) -> int:
 
 
 def router_topk(x: torch.Tensor, w_router: torch.Tensor, E: int, k: int, norm_topk: bool,
-                split: Optional[Tuple[torch.Tensor, Optional[torch.Tensor]]] = None, scoring: str = "softmax"
-                ) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
+                split: Optional[Tuple[torch.Tensor, Optional[torch.Tensor]]] = None, scoring: str = "softmax",
+                bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
     """Router logits (float32), softmax, top-k.  Rows of `w_router` beyond E give raw
-    logits back (`extra`, [T, rows - E]).  Returns (idx int32 [T, k], weights float32 [T, k], extra).
+    logits back (`extra`, [T, rows - E]).  `bias` (float32 [E]) is added to the experts' logits.  Returns (idx int32 [T, k], weights float32 [T, k], extra).
 
     With many bfloat16 rows and a `split` of the matrix (see `split_router`) the logits come
     from tensor-core products with float32 sums; otherwise from the float32 CUDA-core kernel."""
     _chk(x, "x"); _chk(w_router, "w_router", torch.float32)
+    if bias is not None:
+        _chk(bias, "bias", torch.float32)
     T, H = x.shape
     extra = w_router.shape[0] - E
     idx = torch.empty((T, k), dtype=torch.int32, device=x.device)
@@ -827,11 +842,11 @@ def router_topk(x: torch.Tensor, w_router: torch.Tensor, E: int, k: int, norm_to
             _skinny(split[1], H, x, 0, low, rows, T, H, 1, rows, None, None, 1, False)
             logits_t += low
         _lib.call("nf_router_select", _p(logits_t), c_longlong(1), c_longlong(T), c_int(T), c_int(E),
-                  c_int(extra), c_int(k), c_int(_route_flags(norm_topk, scoring)), _p(idx), _p(wts), _p(ext), _stream())
+                  c_int(extra), c_int(k), c_int(_route_flags(norm_topk, scoring)), _p(idx), _p(wts), _p(ext), _p(bias), _stream())
         return idx, wts, ext
     logits = torch.empty((T, E + extra), dtype=torch.float32, device=x.device)
     _lib.call("nf_router_topk", _p(x), _p(w_router), c_int(T), c_int(H), c_int(E), c_int(extra),
-              c_int(k), c_int(_route_flags(norm_topk, scoring)), _p(logits), _p(idx), _p(wts), _p(ext),
+              c_int(k), c_int(_route_flags(norm_topk, scoring)), _p(logits), _p(idx), _p(wts), _p(ext), _p(bias),
               c_int(_dt(x)), _stream())
     return idx, wts, ext
 
@@ -854,7 +869,8 @@ _TICKETS = {}
 
 
 def route(x: torch.Tensor, w_router: torch.Tensor, E: int, k: int, norm_topk: bool,
-          split: Optional[Tuple[torch.Tensor, Optional[torch.Tensor]]] = None, scoring: str = "softmax"):
+          split: Optional[Tuple[torch.Tensor, Optional[torch.Tensor]]] = None, scoring: str = "softmax",
+          bias: Optional[torch.Tensor] = None):
     """Routing of a step: `router_topk` and `moe_plan` together -> (idx, weights, extra, plan).
 
     Up to `TUNING["router_fused_max_rows"]` rows this is one launch: blocks compute the
@@ -862,8 +878,10 @@ def route(x: torch.Tensor, w_router: torch.Tensor, E: int, k: int, norm_topk: bo
     _chk(x, "x"); _chk(w_router, "w_router", torch.float32)
     T, H = x.shape
     if T == 0 or T > TUNING["router_fused_max_rows"]:
-        idx, wts, ext = router_topk(x, w_router, E, k, norm_topk, split=split, scoring=scoring)
+        idx, wts, ext = router_topk(x, w_router, E, k, norm_topk, split=split, scoring=scoring, bias=bias)
         return idx, wts, ext, moe_plan(idx, E)
+    if bias is not None:
+        _chk(bias, "bias", torch.float32)
     dev = x.device
     extra = w_router.shape[0] - E
     idx = torch.empty((T, k), dtype=torch.int32, device=dev)
@@ -879,14 +897,14 @@ def route(x: torch.Tensor, w_router: torch.Tensor, E: int, k: int, norm_topk: bo
         # one thread-block cluster: logits meet selection and plan in distributed shared memory
         _lib.call("nf_router_cluster", _p(x), _p(w_router), c_int(T), c_int(H), c_int(E), c_int(extra), c_int(k),
                   c_int(_route_flags(norm_topk, scoring)), None, _p(idx), _p(wts), _p(ext), _p(offsets), _p(order),
-                  _p(inv), _p(active), c_int(active.numel()), c_int(_dt(x)), _stream())
+                  _p(inv), _p(active), c_int(active.numel()), _p(bias), c_int(_dt(x)), _stream())
         return idx, wts, ext, MoePlan(offsets, order, inv, E, T, k, active)
     key = str(dev)
     if key not in _TICKETS:
         _TICKETS[key] = torch.zeros((1,), dtype=torch.int32, device=dev)
     _lib.call("nf_router_fused", _p(x), _p(w_router), c_int(T), c_int(H), c_int(E), c_int(extra), c_int(k),
               c_int(_route_flags(norm_topk, scoring)), _p(logits), _p(idx), _p(wts), _p(ext), _p(offsets), _p(order),
-              _p(inv), _p(active), c_int(active.numel()), _p(_TICKETS[key]), c_int(_dt(x)), _stream())
+              _p(inv), _p(active), c_int(active.numel()), _p(_TICKETS[key]), _p(bias), c_int(_dt(x)), _stream())
     return idx, wts, ext, MoePlan(offsets, order, inv, E, T, k, active)
 
 
@@ -1119,7 +1137,7 @@ def moe_experts(x: torch.Tensor, w13, w2, plan: MoePlan, k: int,
               c_longlong(w2.group_stride), _p(act), _p(y), c_int(T * k), c_int(T), c_int(H), c_int(inner),
               c_int(w13.groups), c_int(k), _p(plan.offsets), _p(plan.order), _p(plan.active),
               c_int(plan.active.numel()), _p(_stream_work(x.device)), c_int(q),
-              c_int(TUNING["moe_stream_smem_kb"] * 1024), None, c_int(0), c_int(0), None, None, None, None, None,
+              c_int(TUNING["moe_stream_smem_kb"] * 1024), None, c_int(0), c_int(0), None, None, None, None, None, None,
               None, c_longlong(0), None, c_longlong(0), c_int(0), None, None, c_int(kind), c_float(limit),
               c_float(alpha), _stream())
     return y
@@ -1162,7 +1180,8 @@ def can_route_and_run_experts(x: torch.Tensor, w_router: torch.Tensor, w13, w2, 
 
 
 def route_and_run_experts(x: torch.Tensor, w_router: torch.Tensor, E: int, k: int, norm_topk: bool, w13, w2,
-                          shared: Optional[Tuple[PackedWeights, PackedWeights]] = None, act=None):
+                          shared: Optional[Tuple[PackedWeights, PackedWeights]] = None, act=None,
+                          bias: Optional[torch.Tensor] = None):
     """`route` and `moe_experts` in the one persistent launch: its CTAs compute the router logits
     between them, the one that finishes last selects and writes the plan, and all go on to the
     experts' products.  Returns (idx, weights, extra, plan, y) as the two calls would.
@@ -1177,6 +1196,8 @@ def route_and_run_experts(x: torch.Tensor, w_router: torch.Tensor, E: int, k: in
     q = _stream_items(x, w13, w2, E, k, routes=True, shared_chunks=chunks)
     if not q:
         raise ValueError("route_and_run_experts: the step does not fit the launch")
+    if bias is not None:
+        _chk(bias, "bias", torch.float32)
     T, H = x.shape
     dev = x.device
     inner = w13.n_features
@@ -1200,7 +1221,7 @@ def route_and_run_experts(x: torch.Tensor, w_router: torch.Tensor, E: int, k: in
               c_longlong(w2.group_stride), _p(act), _p(y), c_int(T * k), c_int(T), c_int(H), c_int(inner),
               c_int(E), c_int(k), _p(offsets), _p(order), _p(active), c_int(active.numel()),
               _p(_stream_work(dev)), c_int(q), c_int(TUNING["moe_stream_smem_kb"] * 1024), _p(w_router),
-              c_int(extra), c_int(1 if norm_topk else 0), _p(logits), _p(idx), _p(wts), _p(ext), _p(inv),
+              c_int(extra), c_int(1 if norm_topk else 0), _p(logits), _p(idx), _p(wts), _p(ext), _p(inv), _p(bias),
               _p(s13.data) if chunks else None, c_longlong(s13.group_stride if chunks else 0),
               _p(s2.data) if chunks else None, c_longlong(s2.group_stride if chunks else 0), c_int(chunks),
               _p(cw), _p(cinv), c_int(kind), c_float(limit), c_float(alpha), _stream())
@@ -1368,6 +1389,51 @@ def routed_scaled_norm_add(h: torch.Tensor, y: torch.Tensor, inv: torch.Tensor, 
     return out
 
 
+def residual_norm(h: torch.Tensor, weight: Optional[torch.Tensor], eps: float, out: Optional[torch.Tensor],
+                  a: Optional[torch.Tensor] = None, scale_a: float = 1.0, b: Optional[torch.Tensor] = None, scale_b: float = 1.0,
+                  routed=None, bias: Optional[torch.Tensor] = None, inner_weight: Optional[torch.Tensor] = None,
+                  inner_eps: float = 0.0, rows: Optional[torch.Tensor] = None) -> None:
+    """What lies between two sublayers with a norm before and after each (float32 stream h [T, W], in place):
+
+        d = scale_a * a + scale_b * b + sum_j wts[t, j] * y[inv[t * k + j]] + bias
+        h += d / rms(d) * inner_weight        (`inner_weight` None: h += d)
+        out = h / rms(h) * weight             (`weight` None: h itself), in `out`'s type
+
+    a, b [T, W] and `routed` = (y, inv, wts or None, k) are each optional and of the engine's type (that of `out`).
+    With `rows`, out[r] belongs to row rows[r] and h is left as it is.  `out` (or None) may be a range of columns of
+    wider rows."""
+    _chk(h, "h", torch.float32)
+    for t, n in ((weight, "weight"), (bias, "bias"), (inner_weight, "inner_weight")):
+        if t is not None:
+            _chk(t, n, torch.float32)
+    dtype = out.dtype if out is not None else None
+    y = inv = wts = None
+    k = 0
+    if routed is not None:
+        y, inv, wts, k = routed
+        _chk(inv, "inv", torch.int32)
+        if wts is not None:
+            _chk(wts, "wts", torch.float32)
+    for t, n in ((a, "a"), (b, "b"), (y, "y")):
+        if t is not None:
+            dtype = dtype or t.dtype
+            _chk(t, n, dtype)
+            if n != "y" and t.shape != h.shape:
+                raise ValueError(f"residual_norm: {n} does not have the stream's shape")
+    R, ldo = h.shape[0], h.shape[1]
+    if rows is not None:
+        _chk(rows, "rows", torch.int32)
+        R = rows.numel()
+    if out is not None:
+        _chk(out, "out", contiguous=False)
+        ldo = out.stride(0)
+        if out.shape != (R, h.shape[1]) or out.stride(1) != 1:
+            raise ValueError("residual_norm: out does not have the rows' shape")
+    _lib.call("nf_residual_norm", _p(h), _p(a), c_float(scale_a), _p(b), c_float(scale_b), _p(y), _p(inv), _p(wts), c_int(k),
+              _p(bias), _p(inner_weight), c_float(inner_eps), _p(rows), _p(weight), c_float(eps), _p(out), c_int(ldo), c_int(R),
+              c_int(h.shape[1]), c_int(_DT[dtype or torch.float32]), _stream())
+
+
 def mean_of_rmsnorms(xs, ws, eps: float) -> torch.Tensor:
     """float32 [T, W]: the mean over m of (xs[m] / rms(xs[m])) * ws[m]; one to four inputs of equal shape."""
     n = len(xs)
@@ -1508,6 +1574,38 @@ def mlstm_gates(src: torch.Tensor, q_col0: int, k_col0: int, q_scale: float, pre
     return gates
 
 
+DELTA_RULE_MAX_DIM = 256
+
+
+def delta_rule(qkv: torch.Tensor, q_col0: int, k_col0: int, v_col0: int, ab: torch.Tensor, a_col0: int, b_col0: int,
+               dt_bias: torch.Tensor, A_log: torch.Tensor, q_scale: float, state: torch.Tensor, state_off: int, ctx,
+               heads: int, kv_heads: int, D: int, V: int) -> torch.Tensor:
+    """The gated delta rule over a step's rows, request by request, from and into each request's state (float32
+    [slots, ...], the [heads, V, D] block starting at element `state_off`): with g = exp(-exp(A_log) softplus(a +
+    dt_bias)) and beta = sigmoid(b) a row and head,
+
+        S <- g S,  u = beta (v - S^T k),  S <- S + k u^T,  o = S^T q.
+
+    q and k (kv_heads x D) and v (heads x V) are columns of `qkv`; q and k are made unit vectors (x / sqrt(sum(x^2) +
+    1e-6)) and q is multiplied by `q_scale`; head h uses q/k head h // (heads / kv_heads).  a and b are columns of
+    `ab`.  Returns o float32 [T, heads * V]."""
+    _chk(qkv, "qkv"); _chk(ab, "ab", qkv.dtype); _chk(state, "state", torch.float32)
+    _chk(dt_bias, "dt_bias", torch.float32); _chk(A_log, "A_log", torch.float32)
+    T = qkv.shape[0]
+    out = torch.empty((T, heads * V), dtype=torch.float32, device=qkv.device)
+    vectors = records = None
+    rows = int(ctx.max_rows_per_seg)
+    if rows > 1:
+        vectors = torch.empty((T, kv_heads, 2, (D + 3) // 4 * 4), dtype=torch.float32, device=qkv.device)
+        records = torch.empty((T, heads, int(_lib.load().nf_delta_rule_record())), dtype=torch.float32, device=qkv.device)
+    _lib.call("nf_delta_rule", _p(qkv), c_int(qkv.shape[1]), c_int(q_col0), c_int(k_col0), c_int(v_col0), _p(ab),
+              c_int(ab.shape[1]), c_int(a_col0), c_int(b_col0), _p(dt_bias), _p(A_log), c_float(q_scale),
+              c_void_p(state.data_ptr() + 4 * state_off), c_longlong(state.stride(0)), _p(ctx.seg_row0), _p(ctx.seg_slot),
+              _p(vectors), _p(records), _p(out), c_int(ctx.S), c_int(rows), c_int(heads), c_int(kv_heads), c_int(D), c_int(V),
+              c_int(_dt(qkv)), _stream())
+    return out
+
+
 # ---------------------------------------------------------------------------------------
 # state-space mixer
 # ---------------------------------------------------------------------------------------
@@ -1530,7 +1628,7 @@ def causal_conv_silu(src: torch.Tensor, col0: int, C: int, taps: torch.Tensor, b
     out = torch.empty((T, C), dtype=src.dtype, device=src.device)
     _lib.call("nf_causal_conv_silu", _p(src), c_int(ld), c_int(col0), c_int(C), _p(taps), _p(bias), c_int(K),
               _p(state), c_longlong(state.stride(0)), _p(ctx.row_seg), _p(ctx.seg_row0), _p(ctx.seg_slot), _p(out),
-              c_int(T), c_int(ctx.S), c_int(_dt(src)), _stream())
+              c_int(T), c_int(ctx.S), c_int(1 if ctx.all_single else 0), c_int(_dt(src)), _stream())
     return out
 
 

@@ -1,1 +1,1 @@
-from . import qwen2_moe, vekasun, difavik, fetezen, kopadra, pudizen  # noqa: F401  (registration)
+from . import qwen2_moe, vekasun, difavik, fetezen, kopadra, pudizen, nolesun  # noqa: F401  (registration)

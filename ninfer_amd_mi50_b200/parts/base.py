@@ -417,10 +417,58 @@ class PairSum:
     b: torch.Tensor
 
 
+@dataclass
+class ScaledPair:
+    """The outputs of two mixers that ran side by side on one input, still to be added up with fixed factors:
+    ``scale_a * a + scale_b * b (+ bias)``; `bias` float32 [hidden] is a projection's, its mixer's factor included."""
+    a: torch.Tensor
+    scale_a: float
+    b: torch.Tensor
+    scale_b: float
+    bias: Optional[torch.Tensor] = None
+
+
+@dataclass
+class NormedUpdate:
+    """What a block with a norm behind each sublayer leaves pending: the stream is still to grow by
+    ``delta / sqrt(mean(delta^2) + eps) * weight`` (`weight` float32 [hidden]: the norm's times the channel scale).
+    `delta` is a tensor, `RoutedSum`, `ScaledPair` or `BiasedOutput`.  A norm that knows the form (`takes_normed`)
+    works all of it out in its own pass over the stream; `apply` does it on its own."""
+    delta: object
+    weight: torch.Tensor
+    eps: float
+
+    def sources(self) -> Dict[str, object]:
+        """`delta` as the arguments of `kernels.residual_norm`, with the norm it is to pass."""
+        d = self.delta
+        args: Dict[str, object] = {"inner_weight": self.weight, "inner_eps": self.eps}
+        if isinstance(d, RoutedSum):
+            if d.shared is None:
+                args["routed"] = (d.y, d.plan.inv, d.wts, d.plan.top_k)
+                return args
+            d = d.materialize()
+        if isinstance(d, ScaledPair):
+            args.update(a=d.a, scale_a=d.scale_a, b=d.b, scale_b=d.scale_b, bias=d.bias)
+        elif isinstance(d, BiasedOutput):
+            args.update(a=d.y, bias=d.bias)
+        else:
+            args["a"] = d
+        return args
+
+    def apply(self, h: torch.Tensor) -> None:
+        from .. import kernels
+        kernels.residual_norm(h, None, 0.0, None, **self.sources())
+
+
 def summed(delta):
     """`delta` as a tensor (None stays None; a `StreamCopy` means nothing is left to add)."""
     if isinstance(delta, PairSum):
         return (delta.a.to(torch.float32) + delta.b.to(torch.float32)).to(delta.a.dtype)
+    if isinstance(delta, ScaledPair):
+        y = delta.a.to(torch.float32) * delta.scale_a + delta.b.to(torch.float32) * delta.scale_b
+        return (y if delta.bias is None else y + delta.bias).to(delta.a.dtype)
+    if isinstance(delta, NormedUpdate):
+        raise TypeError("an update that is still to be normed is applied to the stream, not read as a sum")
     if isinstance(delta, StreamCopy):
         return None
     if isinstance(delta, BiasedOutput):
@@ -441,6 +489,7 @@ class Norm(Part):
     """
 
     takes_unsummed = False
+    takes_normed = False            # accepts a `NormedUpdate` as `delta`
 
     def add_norm(self, h: torch.Tensor, delta: Optional[torch.Tensor],
                  out_dtype: torch.dtype) -> torch.Tensor:
@@ -548,6 +597,9 @@ class Block(Part):
         stream between layers; the step itself never calls it."""
         if isinstance(pending, StreamCopy):
             return pending
+        if isinstance(pending, NormedUpdate):
+            pending.apply(h)
+            return None
         delta = summed(pending)
         if delta is not None:
             h.add_(delta.to(torch.float32))

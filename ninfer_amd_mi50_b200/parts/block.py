@@ -13,8 +13,8 @@ from typing import List, Optional
 
 import torch
 
-from ..registry import register_part
-from .base import Block, CacheView, FeedForward, Fetch, Mixer, Norm, RoutedSum, StepContext, TensorSpec, summed
+from ..registry import build_part, register_part
+from .base import Block, CacheView, FeedForward, Fetch, Mixer, Norm, NormedUpdate, RoutedSum, StepContext, TensorSpec, summed
 
 
 @register_part("block", "pre_norm")
@@ -207,6 +207,74 @@ class SublayerNormScaledBlock(Block):
                 f, bias = f.y, f.bias
             x = self.norm2.add_scaled_norm(h, f, self.scale2, copy_dtype, bias=bias)
         return StreamCopy(x)
+
+
+@register_part("block", "norms_around_scaled")
+class NormsAroundBlock(Block):
+    """A norm before and after each sublayer, and a learned vector that scales the second one's result per channel:
+
+        h += scale1 * norm1b(mixer(norm1(h)));   h += scale2 * norm2b(feed_forward(norm2(h)))
+
+    The sublayer's output, its norm and scale, the sum and the next norm are one pass over the row: each update is
+    left pending (`NormedUpdate`) for the norm that reads the stream next - this block's second, the next block's
+    first or the model's last.  A layer whose feed-forward is ``"none"`` has the first line only.
+    """
+
+    wants_spec = True
+
+    def __init__(self, norm1: Norm, mixer: Mixer, norm2: Norm, feed_forward: FeedForward, spec=None):
+        if spec is None:
+            raise ValueError("this arrangement has tensors of its own and needs the layer's names")
+        self.norm1, self.mixer, self.norm2, self.feed_forward = norm1, mixer, norm2, feed_forward
+        self.norm1b = build_part("norm", spec.norm, prefix=spec.name_of("norm1b"))
+        self.norm2b = build_part("norm", spec.norm, prefix=spec.name_of("norm2b"))
+        for n in (norm1, norm2, self.norm1b, self.norm2b):
+            if not (n.takes_normed and hasattr(n, "weight") and hasattr(n, "eps")):
+                raise TypeError("the arrangement with norms around its sublayers takes norms that apply a pending normed update")
+        names = dict(spec.names)
+        self.width = norm1.size
+        self.scale_names = (spec.prefix + names.get("scale1", "scale1"), spec.prefix + names.get("scale2", "scale2"))
+        self.weight1 = self.weight2 = None          # the second norms' weights times the channel scales
+
+    @property
+    def has_ff(self) -> bool:
+        return not getattr(self.feed_forward, "absent", False)
+
+    def parts(self):
+        first = (self.norm1, self.mixer, self.norm1b)
+        return first + ((self.norm2, self.feed_forward, self.norm2b) if self.has_ff else ())
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(p.graph_safe for p in self.parts())
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        specs = [s for p in self.parts() for s in p.tensor_specs()]
+        return specs + [TensorSpec(n, (self.width,), role="vector", init="norm") for n in self.scale_names[:2 if self.has_ff else 1]]
+
+    def load(self, fetch: Fetch) -> None:
+        for p in self.parts():
+            p.load(fetch)
+        self.weight1 = (self.norm1b.weight * fetch(self.scale_names[0])).contiguous()
+        self.weight2 = (self.norm2b.weight * fetch(self.scale_names[1])).contiguous() if self.has_ff else None
+
+    def weight_bytes(self) -> int:
+        return sum(p.weight_bytes() for p in self.parts())
+
+    def check_limits(self, dtype, max_context, page_size) -> None:
+        for p in self.parts():
+            p.check_limits(dtype, max_context, page_size)
+
+    def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache: Optional[CacheView],
+                state: Optional[torch.Tensor]):
+        if not isinstance(pending, NormedUpdate):
+            pending = summed(pending)
+        x = self.norm1.add_norm(h, pending, ctx.dtype)
+        update = NormedUpdate(self.mixer.forward(x, ctx, cache, state), self.weight1, self.norm1b.eps)
+        if not self.has_ff:
+            return update
+        x = self.norm2.add_norm(h, update, ctx.dtype)
+        return NormedUpdate(self.feed_forward.forward(x, ctx), self.weight2, self.norm2b.eps)
 
 
 @register_part("block", "hyper_connections")

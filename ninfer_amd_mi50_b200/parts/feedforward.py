@@ -127,14 +127,14 @@ class SparseMoeSwiglu(FeedForward):
                      ("up", "experts.{e}.up_proj.weight"), ("down", "experts.{e}.down_proj.weight"),
                      ("shared_gate", "shared_expert.gate_proj.weight"), ("shared_up", "shared_expert.up_proj.weight"),
                      ("shared_down", "shared_expert.down_proj.weight"), ("shared_router", "shared_expert_gate.weight"),
-                     ("correction", "correction"))
+                     ("correction", "correction"), ("router_bias", "gate.bias"))
 
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, norm_topk_prob: bool,
                  moe_intermediate_size: int, shared_intermediate_size: int, prefix: str,
                  scoring: str = "softmax", weight_on: str = "output", tensor_names=None, activation=None,
                  correction: bool = False, groups=None, identity_experts: int = 0, route_scale: float = 1.0,
-                 shared_gate: bool = True):
-        """Further rules of choice (any of them makes the routing `ruled`; softmax scores, weights on the
+                 shared_gate: bool = True, router_bias: bool = False):
+        """`router_bias`: a float32 vector added to the experts' logits.  Further rules of choice (any of them makes the routing `ruled`; softmax scores, weights on the
         outputs and divided by their sum):
         `correction`: a float32 vector added to the scores for the choice only, not for the weights;
         `groups` (count, keep): the experts form `count` equal groups of neighbours, a group scores as its
@@ -158,6 +158,9 @@ class SparseMoeSwiglu(FeedForward):
             count, keep = self.groups
             if count < 1 or total % count or not 1 <= keep <= count or (total // count) * keep < top_k:
                 raise ValueError(f"{total} experts in {count} groups of which {keep} are kept cannot give {top_k} choices")
+        self.has_router_bias, self.router_bias = bool(router_bias), None
+        if self.has_router_bias and self.ruled:
+            raise ValueError("a bias on the router's logits is not served together with further rules of choice")
         self.correction = None
         if self.activation is not None and shared_intermediate_size > 0:
             raise ValueError("a shared expert is served with the silu-gated activation only")
@@ -196,6 +199,8 @@ class SparseMoeSwiglu(FeedForward):
         specs = [TensorSpec(self._n("router"), (self.num_experts + self.identity_experts, H), role="router")]
         if self.has_correction:
             specs.append(TensorSpec(self._n("correction"), (self.num_experts + self.identity_experts,), role="vector"))
+        if self.has_router_bias:
+            specs.append(TensorSpec(self._n("router_bias"), (self.num_experts,), role="vector"))
         for e in range(self.num_experts):
             specs += [TensorSpec(self._n("gate", e), (I, H)),
                       TensorSpec(self._n("up", e), (I, H)),
@@ -211,6 +216,8 @@ class SparseMoeSwiglu(FeedForward):
     def load(self, fetch: Fetch) -> None:
         p, H, I, E = self.prefix, self.hidden_size, self.moe_intermediate_size, self.num_experts
         router = fetch(self._n("router"))
+        if self.has_router_bias:
+            self.router_bias = fetch(self._n("router_bias")).contiguous()
         if self.has_correction:
             self.correction = fetch(self._n("correction")).contiguous()
         if self.has_shared and self.shared_gate:
@@ -275,7 +282,8 @@ class SparseMoeSwiglu(FeedForward):
                 and kernels.can_route_and_run_experts(x, self.w_router, self.w13, self.w2, E, k, shared=self.ws_packed)):
             # a decode step: routing, the experts' products and the shared expert's are one persistent launch
             idx, wts, gate, plan, y, sum_wts, sum_plan = kernels.route_and_run_experts(
-                x, self.w_router, E, k, self.norm_topk_prob, self.w13, self.w2, shared=self.ws_packed, act=self.activation)
+                x, self.w_router, E, k, self.norm_topk_prob, self.w13, self.w2, shared=self.ws_packed, act=self.activation,
+                bias=self.router_bias)
             if SparseMoeSwiglu.record_routing is not None:
                 SparseMoeSwiglu.record_routing.append(idx.clone())
             return RoutedSum(y, sum_plan, sum_wts, None, None, x.dtype)
@@ -317,7 +325,7 @@ class SparseMoeSwiglu(FeedForward):
             with torch.cuda.stream(side):
                 kernels.chain_break()
                 idx, wts, gate, plan = kernels.route(x, self.w_router, E, k, self.norm_topk_prob,
-                                                     split=self.w_router_split)
+                                                     split=self.w_router_split, bias=self.router_bias)
                 if kernels.moe_uses_gathered_rows(x, self.w13):
                     gathered = kernels.moe_gather(x, plan, k)
             shared = kernels.linear(kernels.linear_swiglu(x, self.ws13), self.ws2)
@@ -325,10 +333,11 @@ class SparseMoeSwiglu(FeedForward):
             kernels.chain_break()
         elif fused:
             idx, wts, gate, plan, y = kernels.route_and_run_experts(x, self.w_router, E, k, self.norm_topk_prob,
-                                                                    self.w13, self.w2, act=self.activation)
+                                                                    self.w13, self.w2, act=self.activation,
+                                                                    bias=self.router_bias)
         else:
             idx, wts, gate, plan = kernels.route(x, self.w_router, E, k, self.norm_topk_prob,
-                                                 split=self.w_router_split)
+                                                 split=self.w_router_split, bias=self.router_bias)
             if fork and late:
                 main, side, shared = start_shared()
         if SparseMoeSwiglu.record_routing is not None:
@@ -375,7 +384,7 @@ class SparseMoeSwiglu(FeedForward):
         weights."""
         E, k = self.num_experts, self.top_k
         idx, wts, gate, plan = kernels.route(x, self.w_router, E, k, self.norm_topk_prob,
-                                             split=self.w_router_split, scoring=self.scoring)
+                                             split=self.w_router_split, scoring=self.scoring, bias=self.router_bias)
         if SparseMoeSwiglu.record_routing is not None:
             SparseMoeSwiglu.record_routing.append(idx.clone())
         if self.weight_on == "input":

@@ -23,10 +23,12 @@ Biases, the norms, the rotation and the gate can each be left out.  Further form
 * `value_position`: the value of token j is turned by j over its dimensions (and cached so), and each head's
   output at position i is turned back by i before the gate, so values enter by their relative position.
 * a rotation whose pairs are neighbours (2i, 2i + 1) instead of halves.
+* `softcap` c: the softmax is over ``c tanh(s(i, j) / c)``.
+* `out_bias`: W_o has a bias, which is left to whoever reads the output next (`BiasedOutput`).
 
-With a window or sigmoid weights, keys and values of unequal sizes, or of a size the head-major kernels do
+With a window, sigmoid weights or capped scores, keys and values of unequal sizes, or of a size the head-major kernels do
 not take, are widened with zeros to one that they take (`row`, a multiple of 16); the zeros add nothing to a
-score, and the matching columns of W_o are zero.
+score, and the matching columns of W_o are zero (or, with a gate, are dropped where it is applied).
 
 The projections that read x
 (q, k, v and the gate) are one matrix, fused at load; its product is taken as float32 sums so that
@@ -42,7 +44,7 @@ import torch
 from .. import kernels
 from ..config.model_config import PartSpec
 from ..registry import build_part, register_part
-from .base import CacheSpec, CacheView, Fetch, Mixer, StepContext, TensorSpec
+from .base import BiasedOutput, CacheSpec, CacheView, Fetch, Mixer, StepContext, TensorSpec
 
 
 @register_part("mixer", "whole_norm_gated_attention")
@@ -51,16 +53,18 @@ class WholeNormGatedAttention(Mixer):
 
     DEFAULT_NAMES = (("q", "q"), ("k", "k"), ("v", "v"), ("gate", "g"), ("out", "o"), ("q_bias", "q.b"),
                      ("k_bias", "k.b"), ("v_bias", "v.b"), ("q_norm", "q.norm"), ("k_norm", "k.norm"),
-                     ("weight_bias", "pb"))
+                     ("weight_bias", "pb"), ("out_bias", "o.b"))
 
     def __init__(self, hidden_size: int, heads: int, kv_heads: int, head_dim: int, value_dim: int, scale: float,
                  eps: float, prefix: str, position: Optional[PartSpec] = None, own_kv: bool = True, bias: bool = True,
                  gate: bool = True, tensor_names=None, norm: bool = True, window: Optional[int] = None,
-                 weights: str = "softmax", value_position: Optional[PartSpec] = None):
+                 weights: str = "softmax", value_position: Optional[PartSpec] = None,
+                 softcap: Optional[float] = None, out_bias: bool = False):
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads do not divide into {kv_heads} groups")
-        if gate and (window or weights != "softmax") and head_dim != value_dim:
-            raise ValueError("an elementwise gate is not served with widened heads")
+        self.softcap = 0.0 if softcap is None else float(softcap)
+        if self.softcap < 0.0 or (self.softcap and weights != "softmax"):
+            raise ValueError(f"softcap={softcap}: a positive cap on the softmax's scores")
         self.hidden_size, self.heads, self.kv_heads = int(hidden_size), int(heads), int(kv_heads)
         self.head_dim, self.value_dim = int(head_dim), int(value_dim)
         self.scale, self.eps, self.prefix = float(scale), float(eps), prefix
@@ -76,14 +80,15 @@ class WholeNormGatedAttention(Mixer):
         # the usual pages (and their kernels) when keys and values are of one size those kernels take
         self.row = self.head_dim
         self.head_major = self.head_dim == self.value_dim and self.head_dim in kernels.SUPPORTED_HEAD_DIMS
-        if not self.head_major and (self.window or self.sigmoid):
+        if not self.head_major and (self.window or self.sigmoid or self.softcap):
             self.row, self.head_major = (max(self.head_dim, self.value_dim) + 15) // 16 * 16, True
             kernels.check_head_dim(self.row)
         # numbers a head of the attention's output: the widened row, or the value's size
         self.o_head = self.row if self.head_major else self.value_dim
         self.names = dict(self.DEFAULT_NAMES)
         self.names.update(dict(tensor_names or ()))
-        self.w_in = self.w_o = self.b_q = self.b_k = self.b_v = self.q_norm = self.k_norm = self.weight_bias = None
+        self.has_out_bias = bool(out_bias)
+        self.w_in = self.w_o = self.b_q = self.b_k = self.b_v = self.b_o = self.q_norm = self.k_norm = self.weight_bias = None
 
     def _n(self, what: str) -> str:
         return self.prefix + self.names[what]
@@ -101,6 +106,8 @@ class WholeNormGatedAttention(Mixer):
         width = {"q": self.q_width, "k": self.k_width, "v": self.v_width}
         if self.has_bias:
             specs += [TensorSpec(self._n(n + "_bias"), (width[n],), role="vector") for n in kv]
+        if self.has_out_bias:
+            specs.append(TensorSpec(self._n("out_bias"), (W,), role="vector"))
         if self.has_norm:
             specs += [TensorSpec(self._n(n + "_norm"), (width[n],), role="vector", init="norm") for n in kv if n != "v"]
         if self.sigmoid:
@@ -110,7 +117,7 @@ class WholeNormGatedAttention(Mixer):
     def load(self, fetch: Fetch) -> None:
         self.w_in = torch.cat([fetch(self._n(n)) for n, _ in self._projections()], dim=0).contiguous()
         self.w_o = fetch(self._n("out"))
-        if self.o_head != self.value_dim:       # the columns of a widened head's zeros
+        if self.o_head != self.value_dim and not self.has_gate:     # the columns of a widened head's zeros (a gate drops them)
             w = self.w_o.new_zeros((self.hidden_size, self.heads, self.o_head))
             w[:, :, :self.value_dim] = self.w_o.view(self.hidden_size, self.heads, self.value_dim)
             self.w_o = w.view(self.hidden_size, self.heads * self.o_head)
@@ -118,6 +125,8 @@ class WholeNormGatedAttention(Mixer):
             self.b_q = fetch(self._n("q_bias"))
             if self.own_kv:
                 self.b_k, self.b_v = fetch(self._n("k_bias")), fetch(self._n("v_bias"))
+        if self.has_out_bias:
+            self.b_o = fetch(self._n("out_bias")).contiguous()
         if self.has_norm:
             self.q_norm = fetch(self._n("q_norm"))
             self.k_norm = fetch(self._n("k_norm")) if self.own_kv else None
@@ -168,12 +177,13 @@ class WholeNormGatedAttention(Mixer):
         elif self.head_major:
             turn = (value_freq, Dv, interleaved) if value_freq is not None else None
             o = kernels.paged_attention(q, H, G, P, cache.pages, cache.block_table, cache.page_size, ctx,
-                                        self.window or 0, self.scale, turn=turn)
+                                        self.window or 0, self.scale, turn=turn, softcap=self.softcap)
         else:
             o = kernels.talking_attention(q, H, G, D, Dv, cache.pages, cache.block_table, cache.page_size, ctx, 0,
                                           self.scale, None, None)
         if value_freq is not None and (self.sigmoid or not self.head_major):
             kernels.turn_back(o, ctx.positions, value_freq, H, Dv, row=self.o_head, interleaved=interleaved)
         if self.has_gate:
-            o = kernels.sigmoid_gate_rows(o, proj, g0)
-        return kernels.linear(o, self.w_o)
+            o = kernels.sigmoid_gate_rows(o, proj, g0, heads=H, Dv=Dv)
+        y = kernels.linear(o, self.w_o)
+        return BiasedOutput(y, self.b_o) if self.has_out_bias else y

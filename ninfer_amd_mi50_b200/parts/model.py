@@ -17,7 +17,8 @@ import torch
 from .. import kernels
 from ..config.model_config import LayerCall, ModelPlan
 from ..registry import build_part, part_class
-from .base import CacheSpec, CacheView, Fetch, PairSum, RoutedSum, StateSpec, StepContext, StreamUpdate, TensorSpec, summed
+from .base import (CacheSpec, CacheView, Fetch, NormedUpdate, PairSum, RoutedSum, StateSpec, StepContext, StreamUpdate, TensorSpec,
+                   summed)
 
 
 class DecoderModel:
@@ -52,6 +53,8 @@ class DecoderModel:
             if call.add_vector is not None and not (
                     call.add_vector[0] in vectors and 0 <= call.add_vector[1] < vectors[call.add_vector[0]]):
                 raise ValueError(f"execution order adds a vector the plan does not have: {call}")
+            if call.project is not None and (call.project not in plan.stream_projections or self.streams > 1):
+                raise ValueError(f"execution order applies a matrix the plan does not have, or to several streams: {call}")
         # cache and state slots: usually one per layer (slot i is layer i's); an order that gives a
         # layer a slot of its own per call names more
         self.num_cache_slots = max([len(self.blocks)] + [c.cache + 1 for c in self.order])
@@ -62,6 +65,7 @@ class DecoderModel:
         # and only meaningful for arrangements that leave nothing pending
         self.probe: Optional[Callable[[int, torch.Tensor], None]] = None
         self.vectors: Dict[str, torch.Tensor] = {}
+        self.projections: Dict[str, torch.Tensor] = {}
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
 
@@ -76,6 +80,7 @@ class DecoderModel:
         specs += self.final_norm.tensor_specs()
         for name, rows in self.plan.stream_vectors:
             specs.append(TensorSpec(name, (rows, H), role="vector"))
+        specs += [TensorSpec(name, (H, 2 * H)) for name in self.plan.stream_projections]
         if not self.plan.tie_word_embeddings:
             specs.append(TensorSpec(self.plan.head_name, (V, H)))
         return specs
@@ -88,6 +93,7 @@ class DecoderModel:
             e.load(fetch)
         self.final_norm.load(fetch)
         self.vectors = {name: fetch(name) for name, _ in self.plan.stream_vectors}
+        self.projections = {name: fetch(name) for name in self.plan.stream_projections}
         self.head = self.embedding if self.plan.tie_word_embeddings else fetch(self.plan.head_name)
 
     def _slot_specs(self, count: int, slot_of, spec_of, what: str) -> list:
@@ -128,7 +134,19 @@ class DecoderModel:
         n = sum(b.weight_bytes() for b in self.blocks) + self.final_norm.weight_bytes()
         n += sum(e.weight_bytes() for e in self.embedding_extras)
         n += sum(v.numel() * 4 for v in self.vectors.values())
+        n += sum(v.numel() * v.element_size() for v in self.projections.values())
         return n + self.head.numel() * self.head.element_size()
+
+    def _project(self, h: torch.Tensor, pending, beside_start: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        """W [x; x0] as the new float32 stream, x being h with what is pending added (in the pass that rounds it to
+        the product's input)."""
+        x = beside_start[:, :self.hidden_size]
+        if isinstance(pending, NormedUpdate):
+            kernels.residual_norm(h, None, 0.0, x, **pending.sources())
+        else:
+            delta = summed(pending)
+            kernels.residual_norm(h, None, 0.0, x, a=None if delta is None else delta.to(x.dtype))
+        return kernels.linear(beside_start, w, out_dtype=torch.float32)
 
     # ---- one pass over the step's rows --------------------------------------------------
     def forward(self, ctx: StepContext,
@@ -145,8 +163,14 @@ class DecoderModel:
                 e.start(self.embedding, self.plan.embedding_scale, h, ctx, state_of(self.extra_state_slot0))
             else:
                 e.add(h, ctx, state_of(self.extra_state_slot0 + i))
+        beside_start = None                          # [x | x0] in the engine's type; the right half is written once
+        if any(call.project is not None for call in self.order):
+            beside_start = torch.empty((ctx.T, 2 * self.hidden_size), dtype=ctx.dtype, device=ctx.device)
+            kernels.residual_norm(h, None, 0.0, beside_start[:, self.hidden_size:])
         pending = None
         for run, call in enumerate(self.order):
+            if call.project is not None:
+                h, pending = self._project(h, pending, beside_start, self.projections[call.project]), None
             if call.add_vector is not None:
                 # (the pending contribution has not been added yet; the sums commute)
                 kernels.add_row_vector(h, self.vectors[call.add_vector[0]][call.add_vector[1]])
@@ -160,6 +184,8 @@ class DecoderModel:
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=ctx.device)
         if isinstance(pending, StreamUpdate) and getattr(self.final_norm, "takes_stream_update", False):
             pass                                     # the norm applies the update in its own pass over the rows
+        elif isinstance(pending, NormedUpdate) and self.final_norm.takes_normed:
+            pass                                     # ... or norms the last sublayer's output in it
         elif isinstance(pending, PairSum) and getattr(self.final_norm, "takes_pair", False):
             pass                                     # ... and adds two contributions in it
         elif not self.final_norm.takes_unsummed or not isinstance(pending, (torch.Tensor, RoutedSum, type(None))):

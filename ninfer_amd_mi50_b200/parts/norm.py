@@ -15,13 +15,14 @@ import torch
 
 from .. import kernels
 from ..registry import register_part
-from .base import Fetch, Norm, PairSum, RoutedSum, TensorSpec, summed
+from .base import Fetch, Norm, NormedUpdate, PairSum, RoutedSum, TensorSpec, summed
 
 
 @register_part("norm", "rms_norm")
 class RmsNorm(Norm):
     graph_safe = True
     takes_unsummed = True
+    takes_normed = True
 
     def __init__(self, size: int, eps: float, prefix: str, weight_name: str = "weight", one_plus: bool = False):
         """`one_plus`: the stored weight lies around zero and 1 + w multiplies.  `weight_name` "":
@@ -62,7 +63,9 @@ class RmsNorm(Norm):
 
     def add_norm(self, h, delta, out_dtype):
         out = torch.empty(h.shape, dtype=out_dtype, device=h.device)
-        if self._fusable(delta, out_dtype, h.shape[0]):
+        if isinstance(delta, NormedUpdate):
+            kernels.residual_norm(h, self.weight, self.eps, out, **delta.sources())
+        elif self._fusable(delta, out_dtype, h.shape[0]):
             # the experts' weighted sum, the residual add and the norm in one kernel
             kernels.moe_combine_add_rmsnorm(delta.y, delta.plan, delta.wts, delta.shared, delta.gate, h, None,
                                             self.weight, self.eps, out)
@@ -72,7 +75,9 @@ class RmsNorm(Norm):
 
     def add_norm_rows(self, h, delta, rows, out_dtype):
         out = torch.empty((rows.numel(), h.shape[1]), dtype=out_dtype, device=h.device)
-        if self._fusable(delta, out_dtype, rows.numel()):
+        if isinstance(delta, NormedUpdate):
+            kernels.residual_norm(h, self.weight, self.eps, out, rows=rows, **delta.sources())
+        elif self._fusable(delta, out_dtype, rows.numel()):
             kernels.moe_combine_add_rmsnorm(delta.y, delta.plan, delta.wts, delta.shared, delta.gate, h, rows,
                                             self.weight, self.eps, out)
         else:

@@ -123,10 +123,10 @@ def split_router(w_router):
     return None
 
 
-def router_topk(x, w_router, E, k, norm_topk, split=None):
+def router_topk(x, w_router, E, k, norm_topk, split=None, bias=None):
     logits = _f(x) @ w_router.T
     extra = logits[:, E:].contiguous() if w_router.shape[0] > E else None
-    p = torch.softmax(logits[:, :E], dim=-1)
+    p = torch.softmax(logits[:, :E] if bias is None else logits[:, :E] + bias, dim=-1)
     T = x.shape[0]
     idx = torch.zeros((T, k), dtype=torch.int32, device=x.device)
     wts = torch.zeros((T, k), dtype=torch.float32, device=x.device)
@@ -160,8 +160,8 @@ def moe_plan(topk_idx, E):
     return MoePlan(mk(offsets), mk(order), mk(inv), E, T, k, mk(act + [-1] * (n_act - len(act))))
 
 
-def route(x, w_router, E, k, norm_topk, split=None):
-    idx, wts, ext = router_topk(x, w_router, E, k, norm_topk)
+def route(x, w_router, E, k, norm_topk, split=None, bias=None):
+    idx, wts, ext = router_topk(x, w_router, E, k, norm_topk, bias=bias)
     return idx, wts, ext, moe_plan(idx, E)
 
 
