@@ -10,6 +10,7 @@
     python bench.py --config fetezen       # the same for the Fetezen design
     python bench.py --config kopadra       # the same for the Kopadra design
     python bench.py --config pudizen       # the same for the Pudizen design
+    python bench.py --config nolesun       # the same for the Nolesun design, beside Difavik and Vekasun too
 
 One JSON line on stdout.  A "step" is one decode step of a batch of 8 requests, each
 holding a context of about 2,048 tokens (the context length of the named configuration's
@@ -217,8 +218,8 @@ def main() -> int:
     ap.add_argument("--steps", type=int, default=64)
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--config", default="a2.7b", choices=sorted(PROFILES) + ["check-fp32", "vekasun", "difavik", "fetezen", "kopadra", "pudizen"])
-    ap.add_argument("--sizes", default="w1024,w2048,w4096", help="vekasun, difavik, fetezen, kopadra, pudizen: named layer sizes, with commas between them")
+    ap.add_argument("--config", default="a2.7b", choices=sorted(PROFILES) + ["check-fp32", "vekasun", "difavik", "fetezen", "kopadra", "pudizen", "nolesun"])
+    ap.add_argument("--sizes", default="w1024,w2048,w4096", help="vekasun, difavik, fetezen, kopadra, pudizen, nolesun: named layer sizes, with commas between them")
     ap.add_argument("--layers", type=int, default=None, help="fewer layers, for a quick look")
     ap.add_argument("--batch", type=int, default=None)
     ap.add_argument("--long-prefill", action="store_true", help="also time prompts of 8,192 and 32,768 tokens")
@@ -241,7 +242,7 @@ def main() -> int:
     K = max(1, args.steps)
     if args.config == "check-fp32":
         return check_fp32(args)
-    if args.config in ("vekasun", "difavik", "fetezen", "kopadra", "pudizen"):
+    if args.config in ("vekasun", "difavik", "fetezen", "kopadra", "pudizen", "nolesun"):
         return compare_designs(args, W, K)
     CONFIG, FULL_LAYERS, model_name, PROMPT, value_batch, point_batches = PROFILES[args.config]
     args.layers = args.layers or FULL_LAYERS

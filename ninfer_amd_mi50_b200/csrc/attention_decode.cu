@@ -82,6 +82,7 @@ decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_s
   constexpr int HC = 8;                 // query heads per tensor-core pass
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int G = Hq / Hkv;
+  const float in2 = CAPPED ? cap_in2(scale, softcap) : 0.f;
   __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // [kSplit][DS]
   __nv_bfloat16* Vs = Ks + kSplit * DS;                             // [kSplit][DS]
   float* sc = reinterpret_cast<float*>(Vs + kSplit * DS);           // [G][kSplit] scores, then p
@@ -199,7 +200,7 @@ decode_attention_split_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_s
       for (int i = 0; i < 4; ++i) {
         const int r = warp * 32 + m * 16 + g + (i >> 1) * 8;
         const int h = h0 + 2 * tq + (i & 1);
-        if (h < G && r >= n0 && r < n1) sc[h * kSplit + r] = CAPPED ? cap_score(c[m][i] * scale, softcap) : c[m][i] * scale;
+        if (h < G && r >= n0 && r < n1) sc[h * kSplit + r] = CAPPED ? cap_score(c[m][i], softcap, in2) : c[m][i] * scale;
       }
   }
   __syncthreads();

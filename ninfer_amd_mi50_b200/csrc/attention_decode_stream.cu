@@ -93,6 +93,7 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tq = lane & 3;
   const int G = Hq / Hkv;
+  const float in2 = CAPPED ? cap_in2(scale, softcap) : 0.f;
   // one CTA an SM with nearly all of its shared memory: the merge kernel's small CTAs fit beside
   // it and are then in place when the last partial result is written
   asm volatile("griddepcontrol.launch_dependents;");
@@ -265,7 +266,7 @@ decode_attention_stream_kernel(const __nv_bfloat16* __restrict__ qkv, int q_row_
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int key = key0 + nb * 8 + 2 * tq + (i & 1);
-          const float sv = CAPPED ? cap_score(s[nb][i] * scale, softcap) : s[nb][i] * scale;
+          const float sv = CAPPED ? cap_score(s[nb][i], softcap, in2) : s[nb][i] * scale;
           const float v = (key >= k_begin && key < k_end) ? sv : -INFINITY;
           s[nb][i] = v;
           if (i < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);

@@ -236,8 +236,10 @@ __device__ __forceinline__ float gated_act(float g, float u, int kind, float lim
 // Forms of the attention kernels: the softmax, weights sigmoid(score + bias) that are not normalised over keys, and
 // the softmax over scores that were capped, score <- cap * tanh(score / cap).
 enum AttentionForm : int { kFormSoftmax = 0, kFormSigmoid = 1, kFormCapped = 2 };
-// cap * tanh(x / cap) as cap - 2 cap / (1 + exp(2 x / cap)): the error is a few float32 roundings of cap itself.
-__device__ __forceinline__ float cap_score(float x, float cap) { return cap - __fdividef(2.f * cap, 1.f + expf(2.f * x / cap)); }
+// cap * tanh(x * scale / cap) as cap - 2 cap / (1 + 2^(x * in2)) with in2 = 2 log2(e) scale / cap: the error is a few
+// float32 roundings of cap itself.
+__device__ __forceinline__ float cap_score(float x, float cap, float in2) { return cap - __fdividef(2.f * cap, 1.f + exp2f(x * in2)); }
+__device__ __forceinline__ float cap_in2(float scale, float cap) { return 2.f * 1.4426950408889634f * scale / cap; }
 
 __device__ __forceinline__ float relu_square(float v) { const float r = fmaxf(v, 0.f); return r * r; }
 __device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.f + erff(v * 0.70710678118654752f)); }

@@ -15,7 +15,7 @@
 //        ck[s] = D(s, t) k_s.k_t  (s < t),   cq[s] = D(s, t) k_s.q_t  (s <= t),   G_t,  beta_t,  D(t, last).
 //    Products of decays, never quotients: a decay near zero does no harm.
 //
-//  * `delta_rule_chunks_kernel`, one CTA a (request, head, 16 value columns), walks the chunks in order.  A column's
+//  * `delta_rule_chunks_kernel`, one CTA a (request, head, 16 or 8 value columns), walks the chunks in order.  A column's
 //    D state entries lie in the registers of LANES lanes, four consecutive entries every 4 * LANES.  With the state
 //    S_0 at a chunk's start the rule for the whole chunk is
 //        u_t = beta_t (v_t - G_t S_0^T k_t - sum_{s<t} ck_t[s] u_s)
@@ -35,6 +35,7 @@ namespace nf {
 
 constexpr int kDrThreads = 128;
 constexpr int kDrChunk = 8;
+constexpr int kDrColumns = 2;                    // value columns a thread of the chunks' kernel works on
 constexpr int kDrRecord = 2 * kDrChunk + 4;      // ck, cq, (G, beta, D(t, last), 0)
 
 __device__ __forceinline__ float dr_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
@@ -161,50 +162,56 @@ __device__ __forceinline__ void dr_store_state(float* sp, int D, int lane, bool 
   }
 }
 
-template <typename T, int EPL, int LANES>        // D <= EPL * LANES
-__global__ void __launch_bounds__(kDrThreads)
+// CP: value columns a thread works on, so that the vectors it reads from shared memory serve several columns (the
+// kernel is bound by those reads).
+template <typename T, int EPL, int LANES, int CP>        // D <= EPL * LANES
+__global__ void __launch_bounds__(kDrThreads / CP)
 delta_rule_chunks_kernel(const float* __restrict__ vectors, const float* __restrict__ records, const T* __restrict__ vsrc,
                          int ld, int v_col0, float* __restrict__ state, long slot_stride, const int* __restrict__ seg_row0,
                          const int* __restrict__ seg_slot, float* __restrict__ out, int H, int G, int D, int DP, int V) {
+  constexpr int NTH = kDrThreads / CP;
   constexpr int COLS = kDrThreads / LANES;
   constexpr int DPAD = EPL * LANES;
-  constexpr int VR = (kDrChunk * COLS + kDrThreads - 1) / kDrThreads;
+  constexpr int VR = (kDrChunk * COLS + NTH - 1) / NTH;
   __shared__ __align__(16) float sq[2][kDrChunk][DPAD];
   __shared__ __align__(16) float sk[2][kDrChunk][DPAD];
   __shared__ __align__(16) float srec[2][kDrChunk][kDrRecord];
   __shared__ float sv[2][kDrChunk][COLS];
   const int seg = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS, grp = head / (H / G);
-  const int tid = threadIdx.x, lane = tid % LANES, cidx = tid / LANES, col = col0 + cidx;
-  const bool live = col < V;
+  const int tid = threadIdx.x, lane = tid % LANES, cidx = tid / LANES * CP;
   // dimensions from DP to DPAD, and rows beyond a short chunk, are read and multiplied by zeros: they stay zero
-  for (int i = tid; i < 2 * kDrChunk * DPAD; i += kDrThreads) { (&sq[0][0][0])[i] = 0.f; (&sk[0][0][0])[i] = 0.f; }
-  for (int i = tid; i < 2 * kDrChunk * kDrRecord; i += kDrThreads) (&srec[0][0][0])[i] = 0.f;
-  for (int i = tid; i < 2 * kDrChunk * COLS; i += kDrThreads) (&sv[0][0][0])[i] = 0.f;
+  for (int i = tid; i < 2 * kDrChunk * DPAD; i += NTH) { (&sq[0][0][0])[i] = 0.f; (&sk[0][0][0])[i] = 0.f; }
+  for (int i = tid; i < 2 * kDrChunk * kDrRecord; i += NTH) (&srec[0][0][0])[i] = 0.f;
+  for (int i = tid; i < 2 * kDrChunk * COLS; i += NTH) (&sv[0][0][0])[i] = 0.f;
   chain_release_if_small();
   chain_wait(vectors, records, vsrc, state);
   const int row0 = seg_row0[seg], rows = seg_row0[seg + 1] - row0;
   if (rows <= 0) return;
-  float* sp = state + (size_t)seg_slot[seg] * slot_stride + ((size_t)head * V + (live ? col : 0)) * D;
+  float* slot = state + (size_t)seg_slot[seg] * slot_stride + (size_t)head * V * D;
   const bool vec = D % 4 == 0 && slot_stride % 4 == 0 && (uintptr_t)state % 16 == 0;
-  float S[EPL];
-  dr_load_state<EPL, LANES>(sp, D, lane, live, vec, S);
+  float S[CP][EPL];
+#pragma unroll
+  for (int c = 0; c < CP; ++c) {
+    const int col = col0 + cidx + c;
+    dr_load_state<EPL, LANES>(slot + (size_t)(col < V ? col : 0) * D, D, lane, col < V, vec, S[c]);
+  }
   __syncthreads();                               // the zeros are in place before the first copies land
   T rv[VR];
   auto fetch = [&](int c0, int b) {
     const int n = min(kDrChunk, rows - c0), pieces = DP / 4;
-    for (int x = tid; x < n * 2 * pieces; x += kDrThreads) {
+    for (int x = tid; x < n * 2 * pieces; x += NTH) {
       const int t = x / (2 * pieces), i = x - t * 2 * pieces;
       const float* src = vectors + ((size_t)(row0 + c0 + t) * G + grp) * 2 * DP + 4 * i;
       dr_cp16(i < pieces ? &sq[b][t][4 * i] : &sk[b][t][4 * (i - pieces)], src);
     }
-    for (int x = tid; x < n * (kDrRecord / 4); x += kDrThreads) {
+    for (int x = tid; x < n * (kDrRecord / 4); x += NTH) {
       const int t = x / (kDrRecord / 4), i = x - t * (kDrRecord / 4);
       dr_cp16(&srec[b][t][4 * i], records + ((size_t)(row0 + c0 + t) * H + head) * kDrRecord + 4 * i);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
 #pragma unroll
     for (int r = 0; r < VR; ++r) {
-      const int x = tid + r * kDrThreads, t = x / COLS, j = x - t * COLS;
+      const int x = tid + r * NTH, t = x / COLS, j = x - t * COLS;
       rv[r] = from_float<T>(0.f);
       if (t < n && col0 + j < V) rv[r] = vsrc[(size_t)(row0 + c0 + t) * ld + v_col0 + (size_t)head * V + col0 + j];
     }
@@ -215,78 +222,97 @@ delta_rule_chunks_kernel(const float* __restrict__ vectors, const float* __restr
     const int n = min(kDrChunk, rows - c0);
 #pragma unroll
     for (int r = 0; r < VR; ++r) {
-      const int x = tid + r * kDrThreads;
+      const int x = tid + r * NTH;
       if (x < kDrChunk * COLS) sv[b][x / COLS][x % COLS] = to_float(rv[r]);
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                             // chunk c0 has landed; everyone is done with the other buffer
     if (n < kDrChunk) {
       // the last, short chunk: rows left over from the chunk before last count nothing (no write, no decay)
-      for (int x = tid; x < (kDrChunk - n) * DPAD; x += kDrThreads) { (&sq[b][n][0])[x] = 0.f; (&sk[b][n][0])[x] = 0.f; }
-      for (int x = tid; x < (kDrChunk - n) * kDrRecord; x += kDrThreads) (&srec[b][n][0])[x] = 0.f;
+      for (int x = tid; x < (kDrChunk - n) * DPAD; x += NTH) { (&sq[b][n][0])[x] = 0.f; (&sk[b][n][0])[x] = 0.f; }
+      for (int x = tid; x < (kDrChunk - n) * kDrRecord; x += NTH) (&srec[b][n][0])[x] = 0.f;
       __syncthreads();
     } else if (c0 + kDrChunk < rows) {
       fetch(c0 + kDrChunk, b ^ 1);
     }
-    float dk[kDrChunk], dq[kDrChunk];
+    float dk[CP][kDrChunk], dq[CP][kDrChunk];
 #pragma unroll
-    for (int t = 0; t < kDrChunk; ++t) dk[t] = dq[t] = 0.f;
+    for (int c = 0; c < CP; ++c)
+#pragma unroll
+      for (int t = 0; t < kDrChunk; ++t) dk[c][t] = dq[c][t] = 0.f;
 #pragma unroll
     for (int e = 0; e < EPL / 4; ++e) {
 #pragma unroll
       for (int t = 0; t < kDrChunk; ++t) {
         const float4 k4 = *reinterpret_cast<const float4*>(&sk[b][t][(e * LANES + lane) * 4]);
         const float4 q4 = *reinterpret_cast<const float4*>(&sq[b][t][(e * LANES + lane) * 4]);
-        dk[t] = fmaf(S[4 * e], k4.x, dk[t]); dk[t] = fmaf(S[4 * e + 1], k4.y, dk[t]);
-        dk[t] = fmaf(S[4 * e + 2], k4.z, dk[t]); dk[t] = fmaf(S[4 * e + 3], k4.w, dk[t]);
-        dq[t] = fmaf(S[4 * e], q4.x, dq[t]); dq[t] = fmaf(S[4 * e + 1], q4.y, dq[t]);
-        dq[t] = fmaf(S[4 * e + 2], q4.z, dq[t]); dq[t] = fmaf(S[4 * e + 3], q4.w, dq[t]);
+#pragma unroll
+        for (int c = 0; c < CP; ++c) {
+          dk[c][t] = fmaf(S[c][4 * e], k4.x, dk[c][t]); dk[c][t] = fmaf(S[c][4 * e + 1], k4.y, dk[c][t]);
+          dk[c][t] = fmaf(S[c][4 * e + 2], k4.z, dk[c][t]); dk[c][t] = fmaf(S[c][4 * e + 3], k4.w, dk[c][t]);
+          dq[c][t] = fmaf(S[c][4 * e], q4.x, dq[c][t]); dq[c][t] = fmaf(S[c][4 * e + 1], q4.y, dq[c][t]);
+          dq[c][t] = fmaf(S[c][4 * e + 2], q4.z, dq[c][t]); dq[c][t] = fmaf(S[c][4 * e + 3], q4.w, dq[c][t]);
+        }
       }
     }
 #pragma unroll
     for (int w = LANES / 2; w > 0; w >>= 1)
 #pragma unroll
-      for (int t = 0; t < kDrChunk; ++t) {
-        dk[t] += __shfl_xor_sync(0xffffffffu, dk[t], w);
-        dq[t] += __shfl_xor_sync(0xffffffffu, dq[t], w);
-      }
-    // the triangle: every lane of a column works it out for itself
-    float u[kDrChunk], o[kDrChunk];
+      for (int c = 0; c < CP; ++c)
+#pragma unroll
+        for (int t = 0; t < kDrChunk; ++t) {
+          dk[c][t] += __shfl_xor_sync(0xffffffffu, dk[c][t], w);
+          dq[c][t] += __shfl_xor_sync(0xffffffffu, dq[c][t], w);
+        }
+    // the triangle: every lane of a column works it out for itself (u takes dk's place, o dq's)
 #pragma unroll
     for (int t = 0; t < kDrChunk; ++t) {
       float rec[kDrRecord];
 #pragma unroll
       for (int i = 0; i < kDrRecord; i += 4) load4(&srec[b][t][i], rec + i);
-      float r = rec[2 * kDrChunk] * dk[t];
 #pragma unroll
-      for (int s = 0; s < t; ++s) r = fmaf(rec[s], u[s], r);
-      u[t] = rec[2 * kDrChunk + 1] * (sv[b][t][cidx] - r);
-      float y = rec[2 * kDrChunk] * dq[t];
+      for (int c = 0; c < CP; ++c) {
+        float r = rec[2 * kDrChunk] * dk[c][t];
 #pragma unroll
-      for (int s = 0; s <= t; ++s) y = fmaf(rec[kDrChunk + s], u[s], y);
-      o[t] = y;
+        for (int s = 0; s < t; ++s) r = fmaf(rec[s], dk[c][s], r);
+        dk[c][t] = rec[2 * kDrChunk + 1] * (sv[b][t][cidx + c] - r);
+        float y = rec[2 * kDrChunk] * dq[c][t];
+#pragma unroll
+        for (int s = 0; s <= t; ++s) y = fmaf(rec[kDrChunk + s], dk[c][s], y);
+        dq[c][t] = y;
+      }
     }
     const float all = srec[b][n - 1][2 * kDrChunk];
 #pragma unroll
-    for (int i = 0; i < EPL; ++i) S[i] *= all;
+    for (int c = 0; c < CP; ++c) {
+#pragma unroll
+      for (int i = 0; i < EPL; ++i) S[c][i] *= all;
+      // lane t of a column stores row t
+      const int col = col0 + cidx + c;
+#pragma unroll
+      for (int t = 0; t < kDrChunk; ++t) {
+        if (t < n && col < V && lane == t % LANES) out[(size_t)(row0 + c0 + t) * H * V + (size_t)head * V + col] = dq[c][t];
+        dk[c][t] *= srec[b][t][2 * kDrChunk + 2];
+      }
+    }
 #pragma unroll
     for (int t = 0; t < kDrChunk; ++t) {
-      const float f = srec[b][t][2 * kDrChunk + 2] * u[t];
 #pragma unroll
       for (int e = 0; e < EPL / 4; ++e) {
         const float4 k4 = *reinterpret_cast<const float4*>(&sk[b][t][(e * LANES + lane) * 4]);
-        S[4 * e] = fmaf(k4.x, f, S[4 * e]); S[4 * e + 1] = fmaf(k4.y, f, S[4 * e + 1]);
-        S[4 * e + 2] = fmaf(k4.z, f, S[4 * e + 2]); S[4 * e + 3] = fmaf(k4.w, f, S[4 * e + 3]);
+#pragma unroll
+        for (int c = 0; c < CP; ++c) {
+          S[c][4 * e] = fmaf(k4.x, dk[c][t], S[c][4 * e]); S[c][4 * e + 1] = fmaf(k4.y, dk[c][t], S[c][4 * e + 1]);
+          S[c][4 * e + 2] = fmaf(k4.z, dk[c][t], S[c][4 * e + 2]); S[c][4 * e + 3] = fmaf(k4.w, dk[c][t], S[c][4 * e + 3]);
+        }
       }
     }
-    // lane t of a column stores row t
-    if (live) {
-#pragma unroll
-      for (int t = 0; t < kDrChunk; ++t)
-        if (t < n && lane == t % LANES) out[(size_t)(row0 + c0 + t) * H * V + (size_t)head * V + col] = o[t];
-    }
   }
-  dr_store_state<EPL, LANES>(sp, D, lane, live, vec, S);
+#pragma unroll
+  for (int c = 0; c < CP; ++c) {
+    const int col = col0 + cidx + c;
+    dr_store_state<EPL, LANES>(slot + (size_t)(col < V ? col : 0) * D, D, lane, col < V, vec, S[c]);
+  }
 }
 
 // Every segment brings one row.
@@ -372,9 +398,9 @@ static int run_delta_rule(const void* qkv, int ld, int q0, int k0, int v0, const
                  H, G, D, DP);
   if (int rc = check_launch("delta_rule_prepare")) return rc;
 #define NF_DR(E, L)                                                                                                   \
-  launch_chained(delta_rule_chunks_kernel<T, E, L>, dim3(S, H, (V + kDrThreads / L - 1) / (kDrThreads / L)), dim3(kDrThreads), 0, \
-                 stream, (const float*)vectors, (const float*)records, (const T*)qkv, ld, v0, state, slot_stride, seg_row0, \
-                 seg_slot, out, H, G, D, DP, V)
+  launch_chained(delta_rule_chunks_kernel<T, E, L, kDrColumns>, dim3(S, H, (V + kDrThreads / L - 1) / (kDrThreads / L)), \
+                 dim3(kDrThreads / kDrColumns), 0, stream, (const float*)vectors, (const float*)records, (const T*)qkv, ld, v0, \
+                 state, slot_stride, seg_row0, seg_slot, out, H, G, D, DP, V)
   if (D <= 32) NF_DR(4, 8); else if (D <= 64) NF_DR(8, 8); else if (D <= 128) NF_DR(16, 8); else NF_DR(16, 16);
 #undef NF_DR
   return check_launch("delta_rule_chunks");

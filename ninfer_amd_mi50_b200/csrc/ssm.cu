@@ -77,6 +77,72 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ src, int lds, int 
   }
 }
 
+// The same for steps of many rows: a thread keeps its channels' taps in registers and walks ROWS consecutive rows with
+// the last K - 1 inputs in hand, so that every input is read once a tile of rows (and the rows of a tile may belong
+// to several requests).  Same sums in the same order.
+template <typename T, int VE, int K, int ROWS>
+__global__ void __launch_bounds__(128)
+causal_conv_silu_rows_kernel(const T* __restrict__ src, int lds, int col0, int C, const float* __restrict__ taps,
+                             const float* __restrict__ bias, const float* __restrict__ state, long slot_stride,
+                             const int* __restrict__ row_seg, const int* __restrict__ seg_row0,
+                             const int* __restrict__ seg_slot, T* __restrict__ out, int T_rows) {
+  const int t0 = blockIdx.x * ROWS;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VE;
+  float w[K][VE], bs[VE];
+  if (c < C) {
+#pragma unroll
+    for (int e = 0; e < VE; e += 4) {
+#pragma unroll
+      for (int j = 0; j < K; ++j) load4(taps + (size_t)j * C + c + e, w[j] + e);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) bs[e + i] = bias ? bias[c + e + i] : 0.f;
+    }
+  }
+  chain_wait(src, state);
+  if (c >= C) return;
+  auto load_row = [&](int r, float* u) {
+    if (VE == 8) load8(reinterpret_cast<const __nv_bfloat16*>(src) + (size_t)r * lds + col0 + c, u);
+    else load4(reinterpret_cast<const float*>(src) + (size_t)r * lds + col0 + c, u);
+  };
+  float u[K][VE];                                  // the last K inputs, oldest first
+  int seg = -1;
+  for (int t = t0; t < min(t0 + ROWS, T_rows); ++t) {
+    const int sg = row_seg[t];
+    if (sg != seg) {                               // a tile's or a request's first row: what came before it
+      seg = sg;
+      const int r0 = seg_row0[sg];
+      const float* st = state + (size_t)seg_slot[sg] * slot_stride;
+#pragma unroll
+      for (int j = 1; j < K; ++j) {                // u[j] is the input K - j tokens back (it moves down below)
+        const int r = t - (K - j);
+        if (r >= r0) {
+          load_row(r, u[j]);
+        } else {
+          const int i = (K - 1) - (r0 - r);
+#pragma unroll
+          for (int e = 0; e < VE; ++e) u[j][e] = i >= 0 ? st[(size_t)i * C + c + e] : 0.f;
+        }
+      }
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < K; ++j)
+#pragma unroll
+      for (int e = 0; e < VE; ++e) u[j][e] = u[j + 1][e];
+    load_row(t, u[K - 1]);
+    float acc[VE];
+#pragma unroll
+    for (int e = 0; e < VE; ++e) {
+      acc[e] = bs[e];
+#pragma unroll
+      for (int j = 0; j < K; ++j) acc[e] = fmaf(w[j][e], u[j][e], acc[e]);
+      acc[e] = acc[e] / (1.f + expf(-acc[e]));
+    }
+    T* o = out + (size_t)t * C + c;
+#pragma unroll
+    for (int e = 0; e < VE; e += 4) store4(o + e, acc + e);
+  }
+}
+
 // The slot's K - 1 rows become the last K - 1 inputs after this step.
 template <typename T>
 __global__ void conv_state_shift_kernel(const T* __restrict__ src, int lds, int col0, int C, int K,
@@ -351,9 +417,15 @@ extern "C" int nf_causal_conv_silu(const void* src, int lds, int col0, int C, co
   launch_chained(causal_conv_silu_kernel<TT, VE, SI>, dim3(T, (C / (VE) + (VE > 1 ? 127 : 255)) / (VE > 1 ? 128 : 256)),  \
                  dim3(VE > 1 ? 128 : 256), 0, stream, (const TT*)src, lds, col0, C, taps, bias, K, state, (long)slot_stride, \
                  row_seg, seg_row0, seg_slot, (TT*)out, T)
+#define NF_CONV_R(TT, VE, KK)                                                                                            \
+  launch_chained(causal_conv_silu_rows_kernel<TT, VE, KK, 16>, dim3((T + 15) / 16, (C / (VE) + 127) / 128), dim3(128), 0,  \
+                 stream, (const TT*)src, lds, col0, C, taps, bias, (const float*)state, (long)slot_stride, row_seg, seg_row0, \
+                 seg_slot, (TT*)out, T)
 #define NF_CONV_T(TT, VE)                                                                                                \
   do {                                                                                                                  \
-    if (vec) { if (single) NF_CONV(TT, VE, true); else NF_CONV(TT, VE, false); }                                        \
+    if (vec && !single && T >= 64 && K >= 2 && K <= 4 && (uintptr_t)taps % 16 == 0) {                                  \
+      if (K == 2) NF_CONV_R(TT, VE, 2); else if (K == 3) NF_CONV_R(TT, VE, 3); else NF_CONV_R(TT, VE, 4);               \
+    } else if (vec) { if (single) NF_CONV(TT, VE, true); else NF_CONV(TT, VE, false); }                                 \
     else { if (single) NF_CONV(TT, 1, true); else NF_CONV(TT, 1, false); }                                              \
     if (K > 1 && !single)                                                                                               \
       launch_chained(conv_state_shift_kernel<TT>, sgrid, dim3(256), 0, stream, (const TT*)src, lds, col0, C, K, state,   \
@@ -361,6 +433,7 @@ extern "C" int nf_causal_conv_silu(const void* src, int lds, int col0, int C, co
   } while (0)
   if (dtype == kF32) NF_CONV_T(float, 4); else NF_CONV_T(__nv_bfloat16, 8);
 #undef NF_CONV_T
+#undef NF_CONV_R
 #undef NF_CONV
   return check_launch("causal_conv_silu");
 }

@@ -6,6 +6,7 @@ every kernel of one step timed by name against its roofline.
     python bench.py --config fetezen
     python bench.py --config kopadra
     python bench.py --config pudizen
+    python bench.py --config nolesun
 
 For each named size a Vekasun model (latent attention and state-space mixers alternating, routed
 experts scored by a sigmoid and weighted on their input) and a Qwen2-MoE model of the same width,
@@ -127,6 +128,25 @@ def pudizen_config(s: dict) -> dict:
             "layers": [dict(m, mlp=mlp) for m in (att, win, lat, att)]}
 
 
+# the Nolesun design at the same sizes: as many key heads as query heads, heads of 128 with half of them turned, the
+# state-space mixer of the Vekasun comparison beside one attention, a delta rule with heads of 128 x 128 (two sharing a
+# query/key head) beside the other, one dense layer as wide as a token's chosen experts together, the middle layers
+# entered once through the loop's matrix
+def nolesun_config(s: dict) -> dict:
+    H = s["heads"]
+    att = {"heads": H, "kv_heads": H, "dim": HEAD_DIM, "vdim": HEAD_DIM, "scale": HEAD_DIM ** -0.5,
+           "rot": {"base": 10000.0, "dims": ROT_DIM}}
+    ssm = {"heads": s["ssm_heads"], "vdim": SSM_HEAD_DIM, "state": s["state"], "groups": 8, "conv": 4, "norm_groups": 8}
+    rule = {"heads": H, "kv_heads": H // 2, "dim": HEAD_DIM, "vdim": HEAD_DIM, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    one = {"type": "parallel", "mixer": {"left": att, "right": ssm, "left_scale": 0.8, "right_scale": 1.2}}
+    two = {"type": "parallel_2", "mixer": {"left": dict(att, softcap=30.0), "right": rule, "left_scale": 0.9, "right_scale": 0.7}}
+    mlps = [{"kind": "dense", "ff": s["top"] * s["ff"]}, moe, moe, moe]
+    return {"architecture": "Nolesun", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "loop": {"start": 1, "stop": 3, "times": 1},
+            "layers": [dict(m, mlp=f) for m, f in zip((one, two, one, two), mlps)]}
+
+
 def qwen2_dense_config(s: dict) -> dict:
     return dict(qwen2_moe_config(s), mlp_only_layers=list(range(LAYERS)), intermediate_size=4 * s["width"] * 2 // 3 // 64 * 64)
 
@@ -221,6 +241,25 @@ def work_models(s: dict, prompt: int, batch: int, context: int, design: str = ""
                 "nf_heads_sigmoid_gate": (T * H * D * 4, 0.0),
                 "nf_embed_rows": (T * W * (2 + 4), 0.0),
                 "nf_pair_hash_embed": (T * W * (2 + 2 + 4), 0.0),
+            }
+        if design == "nolesun":
+            k, ff = s["top"], s["ff"]
+            rule = (H // 2) * D * 2 + H * D                     # q, k, v channels of the delta rule
+            everything = (rows_ctx * 2 * H * D * 2 + 2 * T * H * D * 2, 4.0 * H * D * pairs)
+            own = {
+                "nf_capped_attention_tc": everything,
+                "nf_decode_attention_further": everything,
+                # q, k, v, a and b in, outputs out; the state read and written once a request
+                "nf_delta_rule": (T * ((rule + 2 * H) * 2 + H * D * 4) + 2 * nseg * H * D * D * 4, 6.0 * T * H * D * D),
+                "nf_causal_conv_silu": (T * (C + rule) / 2 * 4, 8.0 * T * (C + rule) / 2),
+                "nf_whole_norm_rope_append": (T * 3 * H * D * (4 + 2), 0.0),
+                "nf_sigmoid_gate_rows": (T * H * D * (2 + 4 + 2), 0.0),
+                "nf_group_rmsnorm_gate": (T * H * D * (4 + 2 + 2), 0.0),
+                # the stream in and out and the next input out; two mixers' outputs, a dense layer's or k experts' in
+                "nf_residual_norm": (T * W * (10 + (4 + (2 + 3 * 2 * k) / 4) / 2), 0.0),
+                "nf_relu_square": (T * k * ff * (4 + 2), 0.0),
+                "nf_add_row_vector": (T * W * 8, 0.0),
+                "nf_embed_rows": (T * W * (2 + 4), 0.0),
             }
         table = {
             # Fetezen: keys and values of the rows' chunks once, queries in and outputs out; both products and the
@@ -349,8 +388,10 @@ def measure(config: dict, prompt: int, batch: int, context: int, steps: int, war
 
 
 DESIGNS = {"vekasun": vekasun_config, "difavik": difavik_config, "fetezen": fetezen_config, "kopadra": kopadra_config,
-           "pudizen": pudizen_config}
-BESIDE = {"pudizen": qwen2_dense_config}            # the Qwen2-MoE model a design stands beside, where it is not the routed one
+           "pudizen": pudizen_config, "nolesun": nolesun_config}
+# the models a design stands beside, where that is not the routed Qwen2-MoE alone
+BESIDE = {"pudizen": (("qwen2_moe", qwen2_dense_config),),
+          "nolesun": (("difavik", difavik_config), ("vekasun", vekasun_config), ("qwen2_moe", qwen2_moe_config))}
 
 
 def run_comparison(sizes, peaks: dict, prompt: int = 2048, batch: int = 8, context: int = 2048, steps: int = 32,
@@ -359,9 +400,9 @@ def run_comparison(sizes, peaks: dict, prompt: int = 2048, batch: int = 8, conte
     result = {}
     for name in sizes:
         s = SIZES[name]
-        models = work_models(s, prompt, batch, context, design)
         entry = {}
-        for which, cfg in ((design, DESIGNS[design](s)), ("qwen2_moe", BESIDE.get(design, qwen2_moe_config)(s))):
+        for which, make in ((design, DESIGNS[design]), *BESIDE.get(design, (("qwen2_moe", qwen2_moe_config),))):
+            cfg, models = make(s), work_models(s, prompt, batch, context, which if which in DESIGNS else design)
             t0 = time.time()
             m = measure(cfg, prompt, batch, context, steps, warmup)
             for ph in ("prefill", "decode"):

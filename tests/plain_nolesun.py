@@ -20,18 +20,21 @@ import torch
 
 F64 = torch.float64
 
-# (generator, size) or None: every projection's output is disturbed by that fraction of itself, which shows the
-# rows whose logits hang on a near-cancellation or on a close choice of experts
+# (generator, size) or None: what a 16-bit engine would round - projections and what enters them, convolutions - is
+# disturbed by that fraction of itself, which shows the rows whose logits hang on a near-cancellation or on a close
+# choice of experts
 NOISE = None
+
+
+def rounded(x: torch.Tensor) -> torch.Tensor:
+    return x if NOISE is None else x * (1.0 + NOISE[1] * torch.randn(x.shape, generator=NOISE[0], dtype=F64))
 
 
 def proj(h: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor] = None) -> torch.Tensor:
     y = h @ w.T
     if b is not None:
         y = y + b
-    if NOISE is not None:
-        y = y * (1.0 + NOISE[1] * torch.randn(y.shape, generator=NOISE[0], dtype=F64))
-    return y
+    return rounded(y)
 
 
 def rms(x: torch.Tensor, eps: float) -> torch.Tensor:
@@ -40,7 +43,7 @@ def rms(x: torch.Tensor, eps: float) -> torch.Tensor:
 
 def norm(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
     """The stored weight lies around zero."""
-    return rms(x, eps) * (1.0 + w)
+    return rounded(rms(x, eps) * (1.0 + w))
 
 
 def silu(x: torch.Tensor) -> torch.Tensor:
@@ -94,7 +97,7 @@ def attention(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: Dict, neig
     o = out.reshape(T, H * Dv)
     if gated:
         o = o * torch.sigmoid(proj(h, w[p + "g"]))
-    return proj(o, w[p + "o"], bias("o"))
+    return proj(rounded(o), w[p + "o"], bias("o"))
 
 
 # ---- recurrences --------------------------------------------------------------------------------
@@ -116,7 +119,7 @@ def state_space(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: Dict, ep
     H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
     inner = H * P
     z, u, dt = torch.split(proj(h, w[p + "in"]), [inner, inner + 2 * G * N, H], dim=1)
-    u = silu(short_conv(u, w[p + "conv"], w[p + "conv.b"]))
+    u = rounded(silu(short_conv(u, w[p + "conv"], w[p + "conv.b"])))
     x, B, C = u[:, :inner].view(T, H, P), u[:, inner:inner + G * N].view(T, G, N), u[:, inner + G * N:].view(T, G, N)
     dt = softplus(dt + w[p + "dt_bias"])
     rate = torch.exp(w[p + "A_log"])
@@ -130,7 +133,7 @@ def state_space(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: Dict, ep
     y = y.reshape(T, inner) * silu(z)
     parts = int(m["norm_groups"])
     y = rms(y.view(T, parts, inner // parts), eps).reshape(T, inner) * w[p + "norm"]
-    return proj(y, w[p + "o"])
+    return proj(rounded(y), w[p + "o"])
 
 
 def unit(x: torch.Tensor) -> torch.Tensor:
@@ -147,7 +150,7 @@ def delta_step(S: torch.Tensor, q, k, v, g, beta) -> Tuple[torch.Tensor, torch.T
 def delta_rule(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: Dict, eps: float) -> torch.Tensor:
     T = h.shape[0]
     H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q, k, v = (silu(short_conv(proj(h, w[p + n]), w[p + n + ".conv"])) for n in ("q", "k", "v"))
+    q, k, v = (rounded(silu(short_conv(proj(h, w[p + n]), w[p + n + ".conv"]))) for n in ("q", "k", "v"))
     q, k, v = unit(q.view(T, G, D)) * D ** -0.5, unit(k.view(T, G, D)), v.view(T, H, V)
     beta = torch.sigmoid(proj(h, w[p + "b"]))
     g = torch.exp(-torch.exp(w[p + "A_log"]) * softplus(proj(h, w[p + "a"]) + w[p + "dt_bias"]))
@@ -158,7 +161,7 @@ def delta_rule(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: Dict, eps
         for t in range(T):
             S, out[t, hd] = delta_step(S, q[t, kh], k[t, kh], v[t, hd], g[t, hd], beta[t, hd])
     o = (rms(out, eps) * w[p + "norm"]).reshape(T, H * V)
-    return proj(o * silu(proj(h, w[p + "g"])), w[p + "o"])
+    return proj(rounded(o * silu(proj(h, w[p + "g"]))), w[p + "o"])
 
 
 def mixer(h, w, p: str, L: Dict, eps: float) -> torch.Tensor:
@@ -186,8 +189,15 @@ def choose(z: torch.Tensor, top: int) -> Tuple[torch.Tensor, torch.Tensor]:
     return idx, torch.softmax(best, dim=-1)
 
 
-def moe(h, w, p: str, f: Dict) -> torch.Tensor:
-    idx, wts = choose(proj(h, w[p + "router"], w[p + "router.b"]), int(f["router"]["top"]))
+def moe(h, w, p: str, f: Dict, forced: Optional[torch.Tensor] = None, record: Optional[list] = None) -> torch.Tensor:
+    """`forced` [T, top]: the experts to use instead of the largest logits' (weighted by the softmax over theirs);
+    `record` receives (logits, experts)."""
+    z = proj(h, w[p + "router"], w[p + "router.b"])
+    idx, wts = choose(z, int(f["router"]["top"]))
+    if forced is not None:
+        idx, wts = forced, torch.softmax(torch.gather(z, 1, forced), dim=-1)
+    if record is not None:
+        record.append((z, idx))
     out = torch.zeros_like(h)
     for e in range(int(f["router"]["experts"])):
         rows, j = torch.nonzero(idx == e, as_tuple=True)
@@ -215,12 +225,14 @@ def enter_pass(x, x0, w, t: int) -> torch.Tensor:
     return proj(torch.cat([x, x0], dim=1), w["loop.in"]) + w["loop.step"][t]
 
 
-def forward(cfg: Dict, weights: Dict[str, torch.Tensor], tokens: List[int]):
-    """-> (logits [T, vocab], streams [layer runs, T, width]) in double precision."""
+def forward(cfg: Dict, weights: Dict[str, torch.Tensor], tokens: List[int], forced: Optional[list] = None,
+            record: Optional[list] = None):
+    """-> (logits [T, vocab], streams [layer runs, T, width]) in double precision.  `forced`: the experts [T, top] of
+    every routed run, in order; `record` receives each routed run's (logits, experts)."""
     w = {k: v.to(F64) for k, v in weights.items()}
     eps = float(cfg["norm"]["eps"])
     x = x0 = w["embed"][torch.tensor(tokens)] * float((cfg.get("embedding") or {}).get("scale", 1.0))
-    streams = []
+    streams, routed = [], 0
     for i, t in layer_runs(cfg):
         L, p = cfg["layers"][i], f"l{i}."
         if t is not None and i == int(cfg["loop"]["start"]):
@@ -230,7 +242,11 @@ def forward(cfg: Dict, weights: Dict[str, torch.Tensor], tokens: List[int]):
         f = L.get("mlp")
         if f:
             h = norm(x, w[p + "norm2"], eps)
-            y = relu2_mlp(h, w, p + "mlp.") if f["kind"] == "dense" else moe(h, w, p + "mlp.", f)
+            if f["kind"] == "dense":
+                y = relu2_mlp(h, w, p + "mlp.")
+            else:
+                y = moe(h, w, p + "mlp.", f, None if forced is None else forced[routed], record)
+                routed += 1
             x = x + norm(y, w[p + "norm2b"], eps) * w[p + "ls2"]
         streams.append(x.clone())
     return norm(x, w["final.norm"], eps) @ w["head"].T, torch.stack(streams)
