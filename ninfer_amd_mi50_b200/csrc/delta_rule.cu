@@ -35,14 +35,14 @@ namespace nf {
 
 constexpr int kDrThreads = 128;
 constexpr int kDrChunk = 8;
-constexpr int kDrColumns = 2;                    // value columns a thread of the chunks' kernel works on
 constexpr int kDrRecord = 2 * kDrChunk + 4;      // ck, cq, (G, beta, D(t, last), 0)
 
 __device__ __forceinline__ float dr_softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float dr_decay(float a, float dt_bias, float A_log) { return expf(-expf(A_log) * dr_softplus(a + dt_bias)); }
 __device__ __forceinline__ float dr_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
-// vectors [T][G][2][DP]: unit q (times q_scale) and unit k, zeros from D to DP; records [T][H][kDrRecord].
+// vectors [T][G][2][DP]: unit q (times q_scale) and unit k, zeros from D to DP (the chunks' kernel's row, DPAD there);
+// records [T][H][kDrRecord].
 template <typename T>
 __global__ void __launch_bounds__(32 * kDrChunk)
 delta_rule_prepare_kernel(const T* __restrict__ qkv, int ld, int q_col0, int k_col0, const T* __restrict__ ab, int ld_ab,
@@ -162,13 +162,12 @@ __device__ __forceinline__ void dr_store_state(float* sp, int D, int lane, bool 
   }
 }
 
-// CP: value columns a thread works on, so that the vectors it reads from shared memory serve several columns (the
-// kernel is bound by those reads).
+// CP: value columns a thread works on; with two, the vectors it reads from shared memory serve both.
 template <typename T, int EPL, int LANES, int CP>        // D <= EPL * LANES
 __global__ void __launch_bounds__(kDrThreads / CP)
 delta_rule_chunks_kernel(const float* __restrict__ vectors, const float* __restrict__ records, const T* __restrict__ vsrc,
                          int ld, int v_col0, float* __restrict__ state, long slot_stride, const int* __restrict__ seg_row0,
-                         const int* __restrict__ seg_slot, float* __restrict__ out, int H, int G, int D, int DP, int V) {
+                         const int* __restrict__ seg_slot, float* __restrict__ out, int H, int G, int D, int V) {
   constexpr int NTH = kDrThreads / CP;
   constexpr int COLS = kDrThreads / LANES;
   constexpr int DPAD = EPL * LANES;
@@ -179,7 +178,7 @@ delta_rule_chunks_kernel(const float* __restrict__ vectors, const float* __restr
   __shared__ float sv[2][kDrChunk][COLS];
   const int seg = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS, grp = head / (H / G);
   const int tid = threadIdx.x, lane = tid % LANES, cidx = tid / LANES * CP;
-  // dimensions from DP to DPAD, and rows beyond a short chunk, are read and multiplied by zeros: they stay zero
+  // rows beyond a short first chunk are read and multiplied by zeros
   for (int i = tid; i < 2 * kDrChunk * DPAD; i += NTH) { (&sq[0][0][0])[i] = 0.f; (&sk[0][0][0])[i] = 0.f; }
   for (int i = tid; i < 2 * kDrChunk * kDrRecord; i += NTH) (&srec[0][0][0])[i] = 0.f;
   for (int i = tid; i < 2 * kDrChunk * COLS; i += NTH) (&sv[0][0][0])[i] = 0.f;
@@ -197,16 +196,20 @@ delta_rule_chunks_kernel(const float* __restrict__ vectors, const float* __restr
   }
   __syncthreads();                               // the zeros are in place before the first copies land
   T rv[VR];
+  const float* vec_src = vectors + ((size_t)row0 * G + grp) * 2 * DPAD;
+  const float* rec_src = records + ((size_t)row0 * H + head) * kDrRecord;
   auto fetch = [&](int c0, int b) {
-    const int n = min(kDrChunk, rows - c0), pieces = DP / 4;
-    for (int x = tid; x < n * 2 * pieces; x += NTH) {
-      const int t = x / (2 * pieces), i = x - t * 2 * pieces;
-      const float* src = vectors + ((size_t)(row0 + c0 + t) * G + grp) * 2 * DP + 4 * i;
-      dr_cp16(i < pieces ? &sq[b][t][4 * i] : &sk[b][t][4 * (i - pieces)], src);
+    const int n = min(kDrChunk, rows - c0);
+    constexpr int PIECES = DPAD / 2, RECS = kDrRecord / 4;       // 16-byte pieces of a row's two vectors, of its record
+#pragma unroll
+    for (int r = 0; r < kDrChunk * PIECES / NTH; ++r) {
+      const int x = tid + r * NTH, t = x / PIECES, i = x % PIECES;
+      if (t < n) dr_cp16(i < PIECES / 2 ? &sq[b][t][4 * i] : &sk[b][t][4 * (i - PIECES / 2)], vec_src + (size_t)(c0 + t) * G * 2 * DPAD + 4 * i);
     }
-    for (int x = tid; x < n * (kDrRecord / 4); x += NTH) {
-      const int t = x / (kDrRecord / 4), i = x - t * (kDrRecord / 4);
-      dr_cp16(&srec[b][t][4 * i], records + ((size_t)(row0 + c0 + t) * H + head) * kDrRecord + 4 * i);
+#pragma unroll
+    for (int r = 0; r < (kDrChunk * RECS + NTH - 1) / NTH; ++r) {
+      const int x = tid + r * NTH, t = x / RECS, i = x % RECS;
+      if (t < n) dr_cp16(&srec[b][t][4 * i], rec_src + (size_t)(c0 + t) * H * kDrRecord + 4 * i);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
 #pragma unroll
@@ -377,6 +380,8 @@ delta_rule_step_kernel(const T* __restrict__ qkv, int ld, int q_col0, int k_col0
   if (live && lane == 0) out[t * H * V + (size_t)head * V + col] = o;
 }
 
+static int g_delta_columns = 0;      // nf_set_delta_rule_columns(): 1 or 2 forces the choice below (measurement)
+
 template <typename T>
 static int run_delta_rule(const void* qkv, int ld, int q0, int k0, int v0, const void* ab, int ld_ab, int a0, int b0,
                           const float* dt_bias, const float* A_log, float q_scale, float* state, long slot_stride,
@@ -397,10 +402,15 @@ static int run_delta_rule(const void* qkv, int ld, int q0, int k0, int v0, const
                  (const T*)qkv, ld, q0, k0, (const T*)ab, ld_ab, a0, b0, dt_bias, A_log, q_scale, seg_row0, vectors, records,
                  H, G, D, DP);
   if (int rc = check_launch("delta_rule_prepare")) return rc;
-#define NF_DR(E, L)                                                                                                   \
-  launch_chained(delta_rule_chunks_kernel<T, E, L, kDrColumns>, dim3(S, H, (V + kDrThreads / L - 1) / (kDrThreads / L)), \
-                 dim3(kDrThreads / kDrColumns), 0, stream, (const float*)vectors, (const float*)records, (const T*)qkv, ld, v0, \
-                 state, slot_stride, seg_row0, seg_slot, out, H, G, D, DP, V)
+  // two columns a thread once there are CTAs enough (one prompt of 2,048 tokens, heads of 128 x 128: with 16 heads 433 us
+  // with one column, 523 with two; with 28 heads 675 and 581)
+  const long ctas = (long)S * H * ((V + kDrThreads / 8 - 1) / (kDrThreads / 8));
+  const bool two = g_delta_columns ? g_delta_columns == 2 : ctas >= 200;
+#define NF_DR(E, L)  do { if (two) NF_DR_C(E, L, 2); else NF_DR_C(E, L, 1); } while (0)
+#define NF_DR_C(E, L, CC)                                                                                             \
+  launch_chained(delta_rule_chunks_kernel<T, E, L, CC>, dim3(S, H, (V + kDrThreads / L - 1) / (kDrThreads / L)),      \
+                 dim3(kDrThreads / CC), 0, stream, (const float*)vectors, (const float*)records, (const T*)qkv, ld, v0, \
+                 state, slot_stride, seg_row0, seg_slot, out, H, G, D, V)
   if (D <= 32) NF_DR(4, 8); else if (D <= 64) NF_DR(8, 8); else if (D <= 128) NF_DR(16, 8); else NF_DR(16, 16);
 #undef NF_DR
   return check_launch("delta_rule_chunks");
@@ -410,12 +420,15 @@ static int run_delta_rule(const void* qkv, int ld, int q0, int k0, int v0, const
 
 using namespace nf;
 
+extern "C" void nf_set_delta_rule_columns(int columns) { g_delta_columns = columns; }
+
 extern "C" int nf_delta_rule_record() { return kDrRecord; }
+extern "C" int nf_delta_rule_row(int D) { return D <= 32 ? 32 : (D <= 64 ? 64 : (D <= 128 ? 128 : 256)); }
 
 // qkv [T, ld]: q (G x D) at q0, k (G x D) at k0, v (H x V) at v0; ab [T, ld_ab]: a (H) at a0, b (H) at b0; all of
 // `dtype`.  dt_bias, A_log float32 [H]; state float32, slot s at state + s * slot_stride: [H][V][D]; out float32
 // [T, H * V].  max_rows: the most rows a segment brings; 1: steps of single rows.  Otherwise vectors float32
-// [T, G, 2, DP], DP = D rounded up to a multiple of 4, and records float32 [T, H, nf_delta_rule_record()] are scratch.
+// [T, G, 2, nf_delta_rule_row(D)] and records float32 [T, H, nf_delta_rule_record()] are scratch.
 extern "C" int nf_delta_rule(const void* qkv, int ld, int q0, int k0, int v0, const void* ab, int ld_ab, int a0, int b0,
                              const float* dt_bias, const float* A_log, float q_scale, float* state, long long slot_stride,
                              const int* seg_row0, const int* seg_slot, float* vectors, float* records, float* out, int S,
@@ -425,7 +438,7 @@ extern "C" int nf_delta_rule(const void* qkv, int ld, int q0, int k0, int v0, co
   NF_REQUIRE(H <= 65535 && (V + 7) / 8 <= 65535 && S <= 65535 && H / G <= 512, "delta rule: too many heads, columns or requests");
   NF_REQUIRE(q0 >= 0 && k0 >= 0 && v0 >= 0 && q0 + G * D <= ld && k0 + G * D <= ld && v0 + H * V <= ld && a0 >= 0 && b0 >= 0 &&
              a0 + H <= ld_ab && b0 + H <= ld_ab, "delta rule: the column ranges leave their rows");
-  const int DP = (D + 3) / 4 * 4;
+  const int DP = nf_delta_rule_row(D);
   NF_REQUIRE(max_rows == 1 || (vectors && records && (uintptr_t)vectors % 16 == 0 && (uintptr_t)records % 16 == 0), "delta rule: prompt portions need their scratch");
   if (dtype == kF32)
     return run_delta_rule<float>(qkv, ld, q0, k0, v0, ab, ld_ab, a0, b0, dt_bias, A_log, q_scale, state, (long)slot_stride, seg_row0, seg_slot, vectors, records, out, S, max_rows, H, G, D, DP, V, stream);

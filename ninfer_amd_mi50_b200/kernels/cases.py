@@ -212,6 +212,36 @@ def case_linear_attention(tokens: int, device, single: bool = False, dim: int = 
                                                               torch.bfloat16))]
 
 
+def case_delta_rule(tokens: int, device, single: bool = False, dim: int = 128):
+    """The gated delta rule (HQ heads of `dim` x 128, two sharing a query/key head) over a prompt of `tokens` rows, or
+    over `tokens` decoded rows of as many requests."""
+    from . import delta_rule
+    G, V = HQ // 2, 128
+    ctx = _one_request(tokens, device, single, 0)
+    width = 2 * G * dim + HQ * V
+    qkv = (torch.randn(tokens, width, device=device) * 0.5).bfloat16()
+    ab = torch.randn(tokens, 2 * HQ, device=device).bfloat16()
+    state = torch.zeros(ctx.S, HQ * V * dim, device=device)
+    zero = torch.zeros(HQ, device=device)
+    return [("delta_rule", lambda: delta_rule(qkv, 0, G * dim, 2 * G * dim, ab, 0, HQ, zero, zero - 3.0, dim ** -0.5, state, 0, ctx,
+                                              HQ, G, dim, V))]
+
+
+def case_capped_attention(tokens: int, device, single: bool = False, context: int = 0, cap: float = 30.0):
+    """Softmax attention over capped scores (HQ query and key heads of 128), and over plain ones: a prompt of `tokens`
+    rows, or `tokens` decoded rows at `context`."""
+    from . import paged_attention
+    D = 128
+    ctx = _one_request(tokens, device, single, context)
+    held = (context + 1) if single else tokens
+    per = (held + PAGE - 1) // PAGE
+    pages = (torch.randn(ctx.S * per + 1, 2, HQ, PAGE, D, device=device) * 0.5).bfloat16()
+    bt = torch.arange(ctx.S * per, dtype=torch.int32, device=device).view(ctx.S, per)
+    q = (torch.randn(tokens, HQ * D, device=device) * 0.5).bfloat16()
+    attend = lambda c: paged_attention(q, HQ, HQ, D, pages, bt, PAGE, ctx, 0, D ** -0.5, softcap=c)
+    return [("capped_attention", lambda: attend(cap)), ("attention", lambda: attend(0.0))]
+
+
 def case_window_attention(tokens: int, device, single: bool = False, context: int = 0, window: int = 1024, keep: int = 4):
     """Softmax attention with a distance slope per head, a window that keeps the first `keep` keys and a head
     gate (HQ query and key heads of 128): a prompt of `tokens` rows, or `tokens` decoded rows at `context`."""
@@ -285,6 +315,10 @@ CASES = {
     "talking_attention_decode8": lambda dev: case_talking_attention(8, dev, True, 2047),
     "linear_attention_prefill": lambda dev: case_linear_attention(2048, dev),
     "linear_attention_decode8": lambda dev: case_linear_attention(8, dev, True),
+    "delta_rule_prefill": lambda dev: case_delta_rule(2048, dev),
+    "delta_rule_decode8": lambda dev: case_delta_rule(8, dev, True),
+    "capped_attention_prefill": lambda dev: case_capped_attention(2048, dev),
+    "capped_attention_decode8": lambda dev: case_capped_attention(8, dev, True, 2048),
     "retention_prefill": lambda dev: case_linear_attention(2048, dev, dim=64, rotary=True),
     "window_attention_prefill": lambda dev: case_window_attention(2048, dev),
     "window_attention_decode8": lambda dev: case_window_attention(8, dev, True, 2048),

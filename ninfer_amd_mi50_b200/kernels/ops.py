@@ -1596,7 +1596,7 @@ def delta_rule(qkv: torch.Tensor, q_col0: int, k_col0: int, v_col0: int, ab: tor
     vectors = records = None
     rows = int(ctx.max_rows_per_seg)
     if rows > 1:
-        vectors = torch.empty((T, kv_heads, 2, (D + 3) // 4 * 4), dtype=torch.float32, device=qkv.device)
+        vectors = torch.empty((T, kv_heads, 2, int(_lib.load().nf_delta_rule_row(c_int(D)))), dtype=torch.float32, device=qkv.device)
         records = torch.empty((T, heads, int(_lib.load().nf_delta_rule_record())), dtype=torch.float32, device=qkv.device)
     _lib.call("nf_delta_rule", _p(qkv), c_int(qkv.shape[1]), c_int(q_col0), c_int(k_col0), c_int(v_col0), _p(ab),
               c_int(ab.shape[1]), c_int(a_col0), c_int(b_col0), _p(dt_bias), _p(A_log), c_float(q_scale),
